@@ -23,6 +23,8 @@
 // channel instead (rows of gate_ld floats, heads side by side vd apart) and the factor is
 // the logit's sigmoid.  `softcap` c > 0: a scaled score s becomes c tanh(s / c) (the
 // hyperbolic tangent as 1 - 2 / (1 + e^(2x)): its error, times c, is far below a score's own).
+// `slopes` (or null): float [n_heads]; slopes[h] times the distance between query and key is
+// taken off the scaled (and capped) score.
 #include "mma_helpers.cuh"
 #include <math.h>
 
@@ -59,7 +61,8 @@ attention_masked_kernel(const bf16* __restrict__ q, int ldq, bf16* __restrict__ 
                         const int* __restrict__ start_pos,
                         int n_heads, int n_kv, int hd, int vd, float scale, int window, int chunk,
                         const float* __restrict__ gate, int n_splits,
-                        float* __restrict__ part_o, float* __restrict__ part_ml, float softcap, int gate_ld) {
+                        float* __restrict__ part_o, float* __restrict__ part_ml, float softcap, int gate_ld,
+                        const float* __restrict__ slopes) {
     chain_release();
     chain_wait();
     constexpr int KCPR = DKP / 8, VCPR = DVP / 8;          // 16-byte chunks per staged row
@@ -150,7 +153,14 @@ attention_masked_kernel(const bf16* __restrict__ q, int ldq, bf16* __restrict__ 
     float m_row[2] = {-INFINITY, -INFINITY};   // running max of scaled scores (log2 domain)
     float l_row[2] = {0.f, 0.f};               // this thread's share of the running sum
     // with a cap the scores are scaled and capped as they leave the product, and only log2(e) is left to multiply
-    const float sl2 = softcap > 0.f ? kLog2e : scale * kLog2e;
+    const float s_in = softcap > 0.f ? kLog2e : scale * kLog2e;
+    // with a slope the scores take their last factor together with the distance's share
+    const float sl2 = slopes ? 1.0f : s_in;
+    float slope[2] = {0.f, 0.f};
+    if (slopes) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) slope[r] = slopes[row_head[r]] * kLog2e;
+    }
     const float cap_in = softcap > 0.f ? scale / softcap : 0.f;
     // what every row of this warp sees of a page without looking closer: the first row's position
     // bounds the keys from above, the last row's first seen key from below
@@ -205,6 +215,16 @@ attention_masked_kernel(const bf16* __restrict__ q, int ldq, bf16* __restrict__ 
                 for (int i = 0; i < 8; ++i) {
 #pragma unroll
                     for (int e = 0; e < 4; ++e) s[i][e] = softcap * tanh_by_exp(s[i][e] * cap_in);
+                }
+            }
+            if (slopes) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int key = j * kPageTokens + i * 8 + t4 * 2 + (e & 1), r = e >> 1;
+                        s[i][e] = fmaf(s[i][e], s_in, slope[r] * (float)(key - row_pos[r]));
+                    }
                 }
             }
             // ---- mask by position (only pages that cross an edge for some row of this warp)
@@ -342,7 +362,8 @@ template <int DKP, int DVP>
 int launch_masked(const bf16* q, int ldq, bf16* out, int ldo, const bf16* kc, const bf16* vc, long long page_stride,
                   const int* block_table, int table_stride, const int* cu_seqlens, const int* slots, const int* start_pos,
                   int n_seqs, int tiles, int n_heads, int n_kv, int hd, int vd, float scale, int window, int chunk,
-                  const float* gate, int n_splits, float* part_o, float* part_ml, float softcap, int gate_ld, cudaStream_t stream) {
+                  const float* gate, int n_splits, float* part_o, float* part_ml, float softcap, int gate_ld,
+                  const float* slopes, cudaStream_t stream) {
     auto kernel = attention_masked_kernel<DKP, DVP>;
     constexpr int smem = masked_smem_bytes<DKP, DVP>();
     static bool configured = false;
@@ -353,7 +374,7 @@ int launch_masked(const bf16* q, int ldq, bf16* out, int ldo, const bf16* kc, co
     }
     return launch_chained(kernel, dim3(tiles * n_splits, n_kv, n_seqs), dim3(128), smem, stream, q, ldq, out, ldo, kc, vc,
                           page_stride, block_table, table_stride, cu_seqlens, slots, start_pos, n_heads, n_kv, hd, vd, scale,
-                          window, chunk, gate, n_splits, part_o, part_ml, softcap, gate_ld);
+                          window, chunk, gate, n_splits, part_o, part_ml, softcap, gate_ld, slopes);
 }
 }  // namespace
 
@@ -392,7 +413,7 @@ GTG_API int gtg_attention_masked_bf16(const void* q, int ldq, void* out, int ldo
                                       const int* cu_seqlens, const int* slots, const int* start_pos, int n_seqs, int max_q_len,
                                       int n_tokens, int n_heads, int n_kv, int hd, int vd, float scale, int window, int chunk,
                                       const float* gate, int n_splits, float* scratch, float softcap, int gate_ld,
-                                      cudaStream_t stream) {
+                                      const float* slopes, cudaStream_t stream) {
     if (n_seqs <= 0 || max_q_len <= 0) return 0;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv || window < 0 || chunk < 0 || n_splits < 1) return kErrBadArgument;
     if (softcap < 0.f || (gate && gate_ld > 0 && gate_ld < n_heads * vd)) return kErrBadArgument;
@@ -409,7 +430,7 @@ GTG_API int gtg_attention_masked_bf16(const void* q, int ldq, void* out, int ldo
 #define GTG_MASKED(DKP, DVP)                                                                                          \
     launch_masked<DKP, DVP>((const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)kc, (const bf16*)vc, page_stride,       \
                             block_table, table_stride, cu_seqlens, slots, start_pos, n_seqs, (int)tiles, n_heads, n_kv, \
-                            hd, vd, scale, window, chunk, gate, n_splits, part_o, part_ml, softcap, gate_ld, stream)
+                            hd, vd, scale, window, chunk, gate, n_splits, part_o, part_ml, softcap, gate_ld, slopes, stream)
     int st;
     if (padded(hd) == 64) st = dvp == 64 ? GTG_MASKED(64, 64) : GTG_MASKED(64, 128);
     else st = dvp == 64 ? GTG_MASKED(128, 64) : GTG_MASKED(128, 128);

@@ -427,6 +427,99 @@ qkv_conv_finish_run_kernel(const float* __restrict__ sums, int ld, const float* 
         __syncwarp();                                        // before the warp's next head overwrites x
     }
 }
+// ---- norms over whole rows of queries and keys ------------------------------------------
+// For mixers whose projection is [ q: n_heads x hd | k: n_kv x hd ], whose values are the
+// keys as projected, and whose queries and keys are normed over all heads at once.  Of a
+// token's row, in float, each stored number rounded once:
+//   * q <- q / sqrt(mean(q^2) + eps) * q_norm * t, the mean over all n_heads x hd numbers;
+//     t = 1 + coef ln(floor((p + 1) / every) + 1) at position p (every 0: t = 1);
+//   * the value row of the cache gets k, the key row k / sqrt(mean(k^2) + eps) * k_norm.
+// A block a token; the row is staged in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(256)
+qk_rows_finish_kernel(const T* __restrict__ qk, int ld, const float* __restrict__ q_norm, const float* __restrict__ k_norm,
+                      float eps, float coef, double every, T* __restrict__ q_out, int ldq, T* __restrict__ kc, T* __restrict__ vc,
+                      long long page_stride, const int* __restrict__ block_table, int table_stride,
+                      const int* __restrict__ token_seq, const int* __restrict__ slots, const int* __restrict__ positions,
+                      int q_w, int k_w, int hd) {
+    chain_release();
+    chain_wait();
+    extern __shared__ __align__(16) float row[];             // q_w + k_w
+    __shared__ float part[2][8];
+    const int n = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const T* src = qk + (size_t)n * ld;
+    const int pos = positions[n];
+    const size_t page_off = (size_t)block_table[(size_t)slots[token_seq[n]] * table_stride + pos / kPageTokens] * page_stride;
+    const size_t at = page_off + (size_t)(pos % kPageTokens) * hd;       // of key/value head 0
+    const int width = q_w + k_w;
+    float sq = 0.f, sk = 0.f;
+    const bool eights = sizeof(T) == 2 && ld % 8 == 0 && q_w % 8 == 0 && hd % 8 == 0 && page_stride % 8 == 0 &&
+                        (reinterpret_cast<uintptr_t>(qk) % 16) == 0 && (reinterpret_cast<uintptr_t>(vc) % 16) == 0 &&
+                        (reinterpret_cast<uintptr_t>(kc) % 16) == 0 && (reinterpret_cast<uintptr_t>(q_out) % 16) == 0 && ldq % 8 == 0;
+    if (eights) {
+        for (int i = tid * 8; i < width; i += 256 * 8) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+            const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
+            float ss = 0.f, f[8];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const float2 g = __bfloat1622float2(h2[e]);
+                f[2 * e] = g.x; f[2 * e + 1] = g.y;
+                ss = fmaf(g.x, g.x, fmaf(g.y, g.y, ss));
+            }
+            reinterpret_cast<float4*>(row + i)[0] = make_float4(f[0], f[1], f[2], f[3]);
+            reinterpret_cast<float4*>(row + i)[1] = make_float4(f[4], f[5], f[6], f[7]);
+            if (i < q_w) sq += ss;
+            else {
+                sk += ss;
+                const int head = (i - q_w) / hd, c = (i - q_w) % hd;
+                *reinterpret_cast<uint4*>(vc + at + (size_t)head * kPageTokens * hd + c) = raw;
+            }
+        }
+    } else {
+        for (int i = tid; i < width; i += 256) {
+            const float x = to_f32<T>(src[i]);
+            row[i] = x;
+            if (i < q_w) sq = fmaf(x, x, sq);
+            else {
+                sk = fmaf(x, x, sk);
+                const int head = (i - q_w) / hd, c = (i - q_w) % hd;
+                vc[at + (size_t)head * kPageTokens * hd + c] = src[i];
+            }
+        }
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) { part[0][warp] = sq; part[1][warp] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { sq += part[0][w]; sk += part[1][w]; }
+    float t = 1.f;
+    if (every > 0.0) t = 1.f + coef * logf((float)(floor(((double)pos + 1.0) / every) + 1.0));
+    const float q_inv = t / sqrtf(sq / (float)q_w + eps), k_inv = 1.f / sqrtf(sk / (float)k_w + eps);
+    if (eights) {
+        for (int i = tid * 8; i < width; i += 256 * 8) {
+            const bool is_q = i < q_w;
+            const float inv = is_q ? q_inv : k_inv;
+            const float* w = is_q ? q_norm + i : k_norm + (i - q_w);
+            float f[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = row[i + e] * inv * __ldg(w + e);
+            uint4 o;
+            __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) oh[e] = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
+            T* dst = is_q ? q_out + (size_t)n * ldq + i : kc + at + (size_t)((i - q_w) / hd) * kPageTokens * hd + (i - q_w) % hd;
+            *reinterpret_cast<uint4*>(dst) = o;
+        }
+    } else {
+        for (int i = tid; i < width; i += 256) {
+            if (i < q_w) q_out[(size_t)n * ldq + i] = from_f32<T>(row[i] * q_inv * q_norm[i]);
+            else kc[at + (size_t)((i - q_w) / hd) * kPageTokens * hd + (i - q_w) % hd] = from_f32<T>(row[i] * k_inv * k_norm[i - q_w]);
+        }
+    }
+}
 }  // namespace
 
 GTG_API int gtg_qkv_finish(int dtype, const float* sums, int ld, const float* bias, const float* cos_sin, int rot,
@@ -521,5 +614,31 @@ GTG_API int gtg_qkv_conv_finish(int dtype, const float* sums, int ld, const floa
     if (dtype == 0) GTG_CONV_FINISH(float);
     if (dtype == 1) GTG_CONV_FINISH(bf16);
 #undef GTG_CONV_FINISH
+    return kErrBadArgument;
+}
+
+GTG_API int gtg_qk_rows_finish(int dtype, const void* qk, int ld, const float* q_norm, const float* k_norm, float eps, float coef,
+                               double every, void* q_out, int ldq, void* kc, void* vc, long long page_stride, const int* block_table,
+                               int table_stride, const int* token_seq, const int* slots, const int* positions, int N, int n_heads,
+                               int n_kv, int hd, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (n_heads <= 0 || n_kv <= 0 || hd <= 0 || !kc || !vc || every < 0.0) return kErrBadArgument;
+    const int q_w = n_heads * hd, k_w = n_kv * hd;
+    if (ld < q_w + k_w || ldq < q_w) return kErrBadArgument;
+    const size_t smem = (size_t)(q_w + k_w) * sizeof(float);
+    if (smem > 200 * 1024) return kErrUnsupported;
+#define GTG_QK_ROWS(T)                                                                                             \
+    do {                                                                                                           \
+        if (smem > 48 * 1024) {                                                                                    \
+            const cudaError_t e = cudaFuncSetAttribute(qk_rows_finish_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                   \
+        }                                                                                                          \
+        return launch_chained(qk_rows_finish_kernel<T>, dim3(N), dim3(256), smem, stream, (const T*)qk, ld, q_norm, k_norm, eps, coef, \
+                              every, (T*)q_out, ldq, (T*)kc, (T*)vc, page_stride, block_table, table_stride, token_seq, slots,   \
+                              positions, q_w, k_w, hd);                                                            \
+    } while (0)
+    if (dtype == 0) GTG_QK_ROWS(float);
+    if (dtype == 1) GTG_QK_ROWS(bf16);
+#undef GTG_QK_ROWS
     return kErrBadArgument;
 }

@@ -24,6 +24,8 @@
 // vd apart, and the factor is the logit's sigmoid.  `softcap` c > 0: a score
 // becomes c tanh(score / c) after the scale.  `sinks` (or null): float [n_heads];
 // exp(sinks[h]) joins head h's softmax denominator, without a key or a value.
+// `slopes` (or null): float [n_heads]; slopes[h] times the distance between the query's
+// position and the key's is taken off head h's score, after the cap.
 #include "common.cuh"
 #include <math.h>
 
@@ -40,7 +42,8 @@ attention_simple_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, i
                         const int* __restrict__ token_seq, const int* __restrict__ slots,
                         const int* __restrict__ positions,
                         int N, int n_heads, int n_kv, int hd, int vd, int vrow, float scale, int window, int chunk,
-                        const float* __restrict__ gate, int gate_ld, float softcap, const float* __restrict__ sinks) {
+                        const float* __restrict__ gate, int gate_ld, float softcap, const float* __restrict__ sinks,
+                        const float* __restrict__ slopes) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long wid = (long long)blockIdx.x * kWarps + warp;
@@ -74,6 +77,7 @@ attention_simple_kernel(const T* __restrict__ q, int ldq, T* __restrict__ out, i
             for (int d = 0; d < hd; ++d) s = fmaf(qs[d], to_f32<T>(kp[d]), s);
             score = s * scale;
             if (softcap > 0.f) score = softcap * tanhf(score / softcap);
+            if (slopes) score = fmaf(-slopes[h], (float)(pos - t), score);
         }
         const float m_new = fmaxf(m, warp_max(score));
         const float p = valid ? expf(score - m_new) : 0.f;
@@ -122,7 +126,8 @@ GTG_API int gtg_attention_simple(int dtype, const void* q, int ldq, void* out, i
                                  const int* block_table, int table_stride,
                                  const int* token_seq, const int* slots, const int* positions,
                                  int N, int n_heads, int n_kv, int hd, int vd, int vrow, float scale, int window, int chunk,
-                                 const float* gate, int gate_ld, float softcap, const float* sinks, cudaStream_t stream) {
+                                 const float* gate, int gate_ld, float softcap, const float* sinks,
+                                 const float* slopes, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (n_heads <= 0 || n_kv <= 0 || n_heads % n_kv != 0 || hd <= 0) return kErrBadArgument;
     if (vd <= 0 || vd > vrow || window < 0 || chunk < 0 || softcap < 0.f) return kErrBadArgument;
@@ -135,7 +140,7 @@ GTG_API int gtg_attention_simple(int dtype, const void* q, int ldq, void* out, i
 #define GTG_SIMPLE(T, PER)                                                                                   \
     attention_simple_kernel<T, PER><<<(unsigned)blocks, kWarps * 32, smem, stream>>>(                            \
         (const T*)q, ldq, (T*)out, ldo, (const T*)kc, (const T*)vc, page_stride, block_table, table_stride,      \
-        token_seq, slots, positions, N, n_heads, n_kv, hd, vd, vrow, scale, window, chunk, gate, gate_ld, softcap, sinks)
+        token_seq, slots, positions, N, n_heads, n_kv, hd, vd, vrow, scale, window, chunk, gate, gate_ld, softcap, sinks, slopes)
     if (dtype == 0) {
         if (vd <= 256) GTG_SIMPLE(float, 8); else if (vd <= 512) GTG_SIMPLE(float, 16); else GTG_SIMPLE(float, 32);
     } else if (dtype == 1) {

@@ -191,9 +191,13 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                             const int* __restrict__ cu_seqlens, const int* __restrict__ slots,
                             const int* __restrict__ start_pos,
                             int n_heads, int n_kv, float scale, int window, int chunk,
-                            const float* __restrict__ gate, float softcap, int gate_ld) {
+                            const float* __restrict__ gate, float softcap, int gate_ld,
+                            const float* __restrict__ slopes) {
     // softcap c > 0: a scaled score s becomes c tanh(s / c) as it leaves tensor memory.  gate_ld > 0: `gate`
     // holds one float logit per output channel (rows of gate_ld, heads side by side) and the factor is its sigmoid.
+    // slopes (or null): float [n_heads]; slopes[h] times the distance between query and key is taken off a score
+    // (after the cap), and the steps run from the nearest keys to the farthest: in the other order every step's
+    // maximum would lie above the one before it and O would be rescaled at every step.
     using S = Shape<HD>;
     constexpr int BK = S::BK;
     extern __shared__ __align__(1024) unsigned char smem[];
@@ -226,6 +230,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (chunk > 0) k_min = max(k_min, (start + tile * BQ) - (start + tile * BQ) % chunk);
     const int j_lo = k_min / kPageTokens, j_hi = k_max / kPageTokens;
     const int n_steps = (j_hi - j_lo + S::kPages) / S::kPages;
+    auto first_page = [&](int i) { return j_lo + S::kPages * (slopes ? n_steps - 1 - i : i); };   // of step i
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -262,8 +267,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                 mbar_expect_tx(kv_full(s), S::kStageBytes);
                 for (int pg = 0; pg < S::kPages; ++pg) {
                     // a page beyond the last one is the step's first page again: finite values under keys that no row sees
-                    const int j = j_lo + S::kPages * i + pg;
-                    const int page = table[j <= j_hi ? j : j_lo + S::kPages * i];
+                    const int j = first_page(i) + pg;
+                    const int page = table[j <= j_hi ? j : first_page(i)];
                     for (int kv = 0; kv < 2; ++kv) {
                         const int row = ((page * 2 + kv) * n_kv + kvh) * kPageTokens;
                         for (int hh = 0; hh < S::kHalves; ++hh)
@@ -318,13 +323,15 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int pos = start + tile * BQ + r;                   // position of this query
         const int seen_from = chunk > 0 ? pos - pos % chunk : 0; // first key of this query's stretch
         const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
-        const float sl2 = softcap > 0.f ? kLog2e : scale * kLog2e;
+        const float s_in = softcap > 0.f ? kLog2e : scale * kLog2e;
+        const float sl2 = slopes ? 1.0f : s_in;                  // with a slope the scores take their factor with the distance's share
+        const float slope = slopes ? slopes[h] * kLog2e : 0.f;
         const float cap_in = softcap > 0.f ? scale / softcap : 0.f;
         float m_run = -INFINITY, l_run = 0.f;
         uint32_t sv[BK];
         bool ok = true;
         for (int i = 0; i < n_steps; ++i) {
-            const int key0 = (j_lo + S::kPages * i) * kPageTokens;   // position of the step's first key
+            const int key0 = first_page(i) * kPageTokens;            // position of the step's first key
             ok = __all_sync(full, mbar_wait<kTest>(s_full, (uint32_t)i & 1u, abort_flag));
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::);
@@ -348,6 +355,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     r = r * fmaf(-y, r, 2.0f);
                     sv[c] = __float_as_uint(fmaf(-twice, r, softcap));
                 }
+            }
+            if (slopes) {
+                const float near = slope * (float)(key0 - pos);
+#pragma unroll
+                for (int c = 0; c < BK; ++c)
+                    sv[c] = __float_as_uint(fmaf(__uint_as_float(sv[c]), s_in, fmaf(slope, (float)c, near)));
             }
             const bool all_visible = (key0 + BK - 1 <= pos) && (window <= 0 || key0 > pos - window) && key0 >= seen_from;
             if (!all_visible) {
@@ -500,7 +513,7 @@ template <int HD, bool kTest>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, bf16* out, int ldo, const int* block_table,
            int table_stride, const int* cu_seqlens, const int* slots, const int* start_pos, int B, int max_q_len,
            int n_heads, int n_kv, float scale, int window, int chunk, const float* gate, float softcap, int gate_ld,
-           cudaStream_t stream) {
+           const float* slopes, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
         cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, kTest>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -511,7 +524,7 @@ int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, bf16* out, int l
     dim3 grid(n_heads, B, (max_q_len + BQ - 1) / BQ);
     return launch_chained(attention_prefill_tc_kernel<HD, kTest>, grid, dim3(kThreads), (size_t)Shape<HD>::kSmemBytes, stream,
                           map_q, map_kv, out, ldo, block_table, table_stride, cu_seqlens, slots, start_pos,
-                          n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld);
+                          n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld, slopes);
 }
 }  // namespace
 
@@ -533,7 +546,7 @@ GTG_API int gtg_attention_prefill_tcgen05(const void* q, int ldq, int n_tokens, 
                                           const int* cu_seqlens, const int* slots, const int* start_pos,
                                           int B, int max_q_len, int n_heads, int n_kv, int hd,
                                           float scale, int window, int chunk, const float* gate, float softcap, int gate_ld,
-                                          cudaStream_t stream) {
+                                          const float* slopes, cudaStream_t stream) {
     if (B <= 0 || max_q_len <= 0) return 0;
     if (window < 0 || chunk < 0 || softcap < 0.f || (gate && gate_ld > 0 && gate_ld < n_heads * hd)) return kErrBadArgument;
     if (hd != 64 && hd != 128) return kErrUnsupported;
@@ -550,7 +563,7 @@ GTG_API int gtg_attention_prefill_tcgen05(const void* q, int ldq, int n_tokens, 
     st = make_map(&map_kv, kc, (long long)n_pages * kv_rows, hd, hd, kPageTokens);
     if (st != 0) return st;
 #define GTG_ARGS map_q, map_kv, (bf16*)out, ldo, block_table, table_stride, cu_seqlens, slots, start_pos, \
-                 B, max_q_len, n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld, stream
+                 B, max_q_len, n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld, slopes, stream
     if (g_test_waits) return hd == 64 ? launch<64, true>(GTG_ARGS) : launch<128, true>(GTG_ARGS);
     return hd == 64 ? launch<64, false>(GTG_ARGS) : launch<128, false>(GTG_ARGS);
 #undef GTG_ARGS

@@ -428,12 +428,14 @@ delta_step_kernel(const float* __restrict__ qk, int ld_qk, const float* __restri
 // ---------------------------------------------- norm per head, weight, sigmoid gate
 // out[n, h, c] = y[n, h, c] / sqrt(mean_c(y[n, h, :]^2) + eps) * weight[c] * sigmoid(gate[n, h, c]):
 // every head of the read-out by its own root mean square, a weight of dv channels that
-// the heads share, and a gate from float logits.  A warp per (token, head).
-template <typename T>
+// the heads share (or one of every head's own: `w_step` dv instead of 0), and a gate from
+// logits of type G.  With `den` (float [n, heads]) a head is divided by its number first.
+// A warp per (token, head).
+template <typename T, typename G>
 __global__ void __launch_bounds__(256)
-head_norm_gate_kernel(const float* __restrict__ y, int ld_y, const float* __restrict__ gate, int ld_gate,
-                      const float* __restrict__ weight, float eps, T* __restrict__ out, int ld_out,
-                      long long n_items, int n_heads, int dv) {
+head_norm_gate_kernel(const float* __restrict__ y, int ld_y, const G* __restrict__ gate, int ld_gate,
+                      const float* __restrict__ weight, int w_step, float eps, const float* __restrict__ den,
+                      T* __restrict__ out, int ld_out, long long n_items, int n_heads, int dv) {
     chain_release();
     chain_wait();
     const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -442,13 +444,18 @@ head_norm_gate_kernel(const float* __restrict__ y, int ld_y, const float* __rest
     const size_t n = (size_t)(item / n_heads);
     const int h = (int)(item % n_heads);
     const float* src = y + n * ld_y + (size_t)h * dv;
+    const float part = den ? 1.0f / den[item] : 1.0f;
     float ss = 0.f;
-    for (int c = lane; c < dv; c += 32) ss = fmaf(src[c], src[c], ss);
-    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
-    const float* gt = gate + n * ld_gate + (size_t)h * dv;
+    for (int c = lane; c < dv; c += 32) {
+        const float v = src[c] * part;
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = part / sqrtf(warp_sum(ss) / (float)dv + eps);
+    const G* gt = gate + n * ld_gate + (size_t)h * dv;
+    const float* w = weight + (size_t)h * w_step;
     T* dst = out + n * ld_out + (size_t)h * dv;
     for (int c = lane; c < dv; c += 32)
-        dst[c] = from_f32<T>(src[c] * inv * weight[c] * (1.0f / (1.0f + expf(-gt[c]))));
+        dst[c] = from_f32<T>(src[c] * inv * w[c] * (1.0f / (1.0f + expf(-to_f32<G>(gt[c])))));
 }
 }  // namespace
 
@@ -535,16 +542,23 @@ GTG_API int gtg_delta_scan(const float* qk, int ld_qk, const float* v, int ld_v,
                           decay, ld_decay, beta, state, out, ld_out, cu_seqlens, slots, n_heads, n_groups, d, dv, R, slices, wide);
 }
 
-GTG_API int gtg_head_norm_gate(int dtype, const float* y, int ld_y, const float* gate, int ld_gate, const float* weight,
-                               float eps, void* out, int ld_out, int N, int n_heads, int dv, cudaStream_t stream) {
+GTG_API int gtg_head_norm_gate(int dtype, int gate_f32, const float* y, int ld_y, const void* gate, int ld_gate, const float* weight,
+                               int w_step, float eps, const float* den, void* out, int ld_out, int N, int n_heads, int dv,
+                               cudaStream_t stream) {
     if (N <= 0) return 0;
     if (n_heads <= 0 || dv <= 0 || ld_y < n_heads * dv || ld_gate < n_heads * dv || ld_out < n_heads * dv) return kErrBadArgument;
+    if (w_step != 0 && w_step != dv) return kErrBadArgument;
     const long long items = (long long)N * n_heads;
     const long long blocks = (items + 7) / 8;
     if (blocks > 0x7fffffffLL) return kErrUnsupported;
-    if (dtype == 0) return launch_chained(head_norm_gate_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, gate,
-                                          ld_gate, weight, eps, (float*)out, ld_out, items, n_heads, dv);
-    if (dtype == 1) return launch_chained(head_norm_gate_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, gate,
-                                          ld_gate, weight, eps, (bf16*)out, ld_out, items, n_heads, dv);
+    if (dtype == 0 && gate_f32)
+        return launch_chained(head_norm_gate_kernel<float, float>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const float*)gate,
+                              ld_gate, weight, w_step, eps, den, (float*)out, ld_out, items, n_heads, dv);
+    if (dtype == 1 && gate_f32)
+        return launch_chained(head_norm_gate_kernel<bf16, float>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const float*)gate,
+                              ld_gate, weight, w_step, eps, den, (bf16*)out, ld_out, items, n_heads, dv);
+    if (dtype == 1)
+        return launch_chained(head_norm_gate_kernel<bf16, bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const bf16*)gate,
+                              ld_gate, weight, w_step, eps, den, (bf16*)out, ld_out, items, n_heads, dv);
     return kErrBadArgument;
 }

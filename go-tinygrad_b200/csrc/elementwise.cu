@@ -10,9 +10,13 @@
 // out[n,:] = table[tokens[n],:] widened to float (the residual stream), times
 // `scale` (1: no scaling, as in model/inference_helpers.go:9-34).  Token ids are validated by the
 // host; an id outside the table is clamped so the kernel never reads outside.
+// `turns` (or null): double [(H + 1) / 2], whole turns a position; channel 2i gets
+// sin(2 pi positions[n] turns[i]) added, channel 2i + 1 the cosine.  The angle is reduced to
+// a fraction of a turn in double, so that far positions lose nothing.
 template <typename T>
 __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict__ table,
-                             float* __restrict__ out, int H, int V, float scale) {
+                             float* __restrict__ out, int H, int V, float scale,
+                             const int* __restrict__ positions, const double* __restrict__ turns) {
     chain_wait();        // the step's metadata is written here or just before: nothing later may start early
     chain_release();
     const int n = blockIdx.x;
@@ -20,16 +24,25 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const T* __restrict
     tok = tok < 0 ? 0 : (tok >= V ? V - 1 : tok);
     const T* src = table + (size_t)tok * H;
     float* dst = out + (size_t)n * H;
-    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f32<T>(src[i]) * scale;
+    if (!turns) {
+        for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = to_f32<T>(src[i]) * scale;
+        return;
+    }
+    const double p = (double)positions[n];
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const double t = p * turns[i >> 1];
+        const float half_turns = (float)(2.0 * (t - rint(t)));
+        dst[i] = to_f32<T>(src[i]) * scale + ((i & 1) ? cospif(half_turns) : sinpif(half_turns));
+    }
 }
 
 GTG_API int gtg_embed(int dtype, const int* tokens, const void* table, float* out,
-                      int N, int H, int V, float scale, cudaStream_t stream) {
+                      int N, int H, int V, float scale, const int* positions, const double* turns, cudaStream_t stream) {
     int st = 0;
     if (N <= 0) return 0;
     const int threads = H >= 1024 ? 256 : 128;
-    if (dtype == 0) st = launch_chained(embed_kernel<float>, dim3(N), dim3(threads), 0, stream, tokens, (const float*)table, out, H, V, scale);
-    else if (dtype == 1) st = launch_chained(embed_kernel<bf16>, dim3(N), dim3(threads), 0, stream, tokens, (const bf16*)table, out, H, V, scale);
+    if (dtype == 0) st = launch_chained(embed_kernel<float>, dim3(N), dim3(threads), 0, stream, tokens, (const float*)table, out, H, V, scale, positions, turns);
+    else if (dtype == 1) st = launch_chained(embed_kernel<bf16>, dim3(N), dim3(threads), 0, stream, tokens, (const bf16*)table, out, H, V, scale, positions, turns);
     else return kErrBadArgument;
     return st;
 }
@@ -38,11 +51,13 @@ GTG_API int gtg_embed(int dtype, const int* tokens, const void* table, float* ou
 // x = residual[r,:] (+ pending[r,:]);  out[i,:] = weight * x * (1/sqrt(mean(x^2)+eps))
 // with r = rows ? rows[i] : i.  Without `rows` the sum is written back to the
 // residual stream.  eps is added to the mean inside the root, and the product
-// is (w*x)*s (backends/simd/vec.go:72-85).
-template <typename T>
+// is (w*x)*s (backends/simd/vec.go:72-85).  kTwo: a second weight over the same row gives
+// a second output, for layers whose sublayers read two norms of one hidden state.
+template <typename T, bool kTwo>
 __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const T* __restrict__ pending,
                                    const float* __restrict__ weight, float eps,
-                                   T* __restrict__ out, const int* __restrict__ rows, int H) {
+                                   T* __restrict__ out, const int* __restrict__ rows, int H,
+                                   const float* __restrict__ weight2, T* __restrict__ out2) {
     chain_release();
     chain_wait();
     extern __shared__ float smem[];
@@ -67,15 +82,22 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const T* __rest
     T* o = out + (size_t)i_out * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x)
         o[i] = from_f32<T>((weight[i] * row[i]) * s);
+    if (kTwo) {
+        T* o2 = out2 + (size_t)i_out * H;
+        for (int i = threadIdx.x; i < H; i += blockDim.x)
+            o2[i] = from_f32<T>((weight2[i] * row[i]) * s);
+    }
 }
 
 // The same for bfloat16 rows whose width is a multiple of 8 and at most 8192:
 // every thread owns 8 consecutive channels, moved with 16- and 32-byte accesses
 // and kept in registers between the sum of squares and the scaling.
+template <bool kTwo>
 __global__ void __launch_bounds__(1024)
 add_rmsnorm_bf16_vec_kernel(float* __restrict__ residual, const bf16* __restrict__ pending,
                             const float* __restrict__ weight, float eps, bf16* __restrict__ out,
-                            const int* __restrict__ rows, int H) {
+                            const int* __restrict__ rows, int H,
+                            const float* __restrict__ weight2, bf16* __restrict__ out2) {
     chain_release();
     chain_wait();
     __shared__ float scratch[33];
@@ -119,39 +141,50 @@ add_rmsnorm_bf16_vec_kernel(float* __restrict__ residual, const bf16* __restrict
         for (int j = 0; j < 4; ++j)
             oh[j] = __floats2bfloat162_rn((w[2 * j] * x[2 * j]) * s, (w[2 * j + 1] * x[2 * j + 1]) * s);
         *reinterpret_cast<uint4*>(out + (size_t)i_out * H + c) = o;
+        if (kTwo) {
+            const float4* wp = reinterpret_cast<const float4*>(weight2 + c);
+            const float4 w0 = wp[0], w1 = wp[1];
+            oh[0] = __floats2bfloat162_rn((w0.x * x[0]) * s, (w0.y * x[1]) * s);
+            oh[1] = __floats2bfloat162_rn((w0.z * x[2]) * s, (w0.w * x[3]) * s);
+            oh[2] = __floats2bfloat162_rn((w1.x * x[4]) * s, (w1.y * x[5]) * s);
+            oh[3] = __floats2bfloat162_rn((w1.z * x[6]) * s, (w1.w * x[7]) * s);
+            *reinterpret_cast<uint4*>(out2 + (size_t)i_out * H + c) = o;
+        }
     }
 }
 
+// weight2 and out2: a second norm of the same rows (both null: none).
 GTG_API int gtg_add_rmsnorm(int dtype, float* residual, const void* pending, const float* weight,
-                            float eps, void* out, const int* rows, int R, int H,
+                            float eps, void* out, const int* rows, int R, int H, const float* weight2, void* out2,
                             cudaStream_t stream) {
     int st = 0;
     if (R <= 0) return 0;
+    if ((weight2 == nullptr) != (out2 == nullptr)) return kErrBadArgument;
     if (dtype == 1 && H % 8 == 0 && H <= 8192 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
-        ((uintptr_t)weight % 16) == 0 && ((uintptr_t)pending % 16) == 0) {
+        ((uintptr_t)weight % 16) == 0 && ((uintptr_t)pending % 16) == 0 && ((uintptr_t)weight2 % 16) == 0 && ((uintptr_t)out2 % 16) == 0) {
         int t = ((H / 8) + 31) / 32 * 32;
-        st = launch_chained(add_rmsnorm_bf16_vec_kernel, dim3(R), dim3(t), 0, stream, residual, (const bf16*)pending, weight, eps, (bf16*)out, rows, H);
+        if (out2)
+            return launch_chained(add_rmsnorm_bf16_vec_kernel<true>, dim3(R), dim3(t), 0, stream, residual, (const bf16*)pending, weight, eps, (bf16*)out, rows, H, weight2, (bf16*)out2);
+        st = launch_chained(add_rmsnorm_bf16_vec_kernel<false>, dim3(R), dim3(t), 0, stream, residual, (const bf16*)pending, weight, eps, (bf16*)out, rows, H, nullptr, nullptr);
         return st;
     }
     int threads = 32;
     while (threads < 1024 && threads * 4 < H) threads *= 2;
     const size_t smem = (size_t)(H + 33) * sizeof(float);
     if (smem > 200 * 1024) return kErrUnsupported;
-    cudaError_t e;
-    if (dtype == 0) {
-        if (smem > 48 * 1024) {
-            e = cudaFuncSetAttribute(add_rmsnorm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-            if (e != cudaSuccess) return (int)e;
-        }
-        st = launch_chained(add_rmsnorm_kernel<float>, dim3(R), dim3(threads), smem, stream, residual, (const float*)pending, weight, eps, (float*)out, rows, H);
-    } else if (dtype == 1) {
-        if (smem > 48 * 1024) {
-            e = cudaFuncSetAttribute(add_rmsnorm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-            if (e != cudaSuccess) return (int)e;
-        }
-        st = launch_chained(add_rmsnorm_kernel<bf16>, dim3(R), dim3(threads), smem, stream, residual, (const bf16*)pending, weight, eps, (bf16*)out, rows, H);
-    } else return kErrBadArgument;
-    return st;
+#define GTG_RMSNORM(T, TWO)                                                                                          \
+    do {                                                                                                             \
+        if (smem > 48 * 1024) {                                                                                      \
+            const cudaError_t e = cudaFuncSetAttribute(add_rmsnorm_kernel<T, TWO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                     \
+        }                                                                                                            \
+        return launch_chained(add_rmsnorm_kernel<T, TWO>, dim3(R), dim3(threads), smem, stream, residual, (const T*)pending, weight, eps, \
+                              (T*)out, rows, H, weight2, (T*)out2);                                                  \
+    } while (0)
+    if (dtype == 0) { if (out2) GTG_RMSNORM(float, true); GTG_RMSNORM(float, false); }
+    if (dtype == 1) { if (out2) GTG_RMSNORM(bf16, true); GTG_RMSNORM(bf16, false); }
+#undef GTG_RMSNORM
+    return kErrBadArgument;
 }
 
 // ------------------------------------------------------------------ SwiGLU
@@ -159,7 +192,7 @@ GTG_API int gtg_add_rmsnorm(int dtype, float* residual, const void* pending, con
 // (backends/simd/vec.go:52-59), or another of the pointwise activations (`kind`).
 // `gu` holds the gate columns then the up columns.
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int M, int I, int kind) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int ldo, int M, int I, int kind) {
     chain_release();
     chain_wait();
     const size_t total = (size_t)M * I;
@@ -170,19 +203,19 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const float g = to_f32<T>(gu[m * 2 * I + i]);
         const float u = to_f32<T>(gu[m * 2 * I + I + i]);
         const float s = kind == 2 ? g / (1.0f + expf(-g)) : activate(g, kind);
-        out[idx] = from_f32<T>(s * u);
+        out[m * ldo + i] = from_f32<T>(s * u);
     }
 }
 
-GTG_API int gtg_swiglu(int dtype, const void* gu, void* out, int M, int I, int kind, cudaStream_t stream) {
+GTG_API int gtg_swiglu(int dtype, const void* gu, void* out, int ldo, int M, int I, int kind, cudaStream_t stream) {
     int st = 0;
     if (M <= 0 || I <= 0) return 0;
-    if (kind < 0 || kind >= kActivations) return kErrBadArgument;
+    if (kind < 0 || kind >= kActivations || ldo < I) return kErrBadArgument;
     const size_t total = (size_t)M * I;
     int blocks = (int)((total + 255) / 256);
     if (blocks > 148 * 16) blocks = 148 * 16;
-    if (dtype == 0) st = launch_chained(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)out, M, I, kind);
-    else if (dtype == 1) st = launch_chained(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, (bf16*)out, M, I, kind);
+    if (dtype == 0) st = launch_chained(swiglu_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)gu, (float*)out, ldo, M, I, kind);
+    else if (dtype == 1) st = launch_chained(swiglu_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, (const bf16*)gu, (bf16*)out, ldo, M, I, kind);
     else return kErrBadArgument;
     return st;
 }
@@ -940,4 +973,122 @@ GTG_API int gtg_scale(float* x, long long total, float factor, cudaStream_t stre
     const long long want = (total + 255) / 256;
     const int blocks = (int)(want > 148 * 16 ? 148 * 16 : want);
     return launch_chained(scale_kernel, dim3(blocks), dim3(256), 0, stream, x, (size_t)total, factor);
+}
+
+// ---- two updates, each normed, averaged and added --------------------------------
+// v = factor * (a / sqrt(mean(a^2) + eps) * wa + b / sqrt(mean(b^2) + eps) * wb), float
+// throughout, per row of two sublayers' outputs; v joins the float rows `residual`, or,
+// where that is null, goes to `out`.
+template <typename T>
+__global__ void normed_pair_kernel(const T* __restrict__ a, const T* __restrict__ b, const float* __restrict__ wa,
+                                   const float* __restrict__ wb, float eps, float factor, float* __restrict__ residual,
+                                   T* __restrict__ out, int H) {
+    chain_release();
+    chain_wait();
+    extern __shared__ float smem[];
+    float* ra = smem;
+    float* rb = smem + H;
+    float* scratch = smem + 2 * H;
+    const size_t base = (size_t)blockIdx.x * H;
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float x = to_f32<T>(a[base + i]), y = to_f32<T>(b[base + i]);
+        ra[i] = x;
+        rb[i] = y;
+        sa += x * x;
+        sb += y * y;
+    }
+    sa = factor / sqrtf(block_sum(sa, scratch) / (float)H + eps);
+    sb = factor / sqrtf(block_sum(sb, scratch) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float v = ra[i] * sa * wa[i] + rb[i] * sb * wb[i];
+        if (residual) residual[base + i] += v;
+        else out[base + i] = from_f32<T>(v);
+    }
+}
+
+// The same for bfloat16 rows of a multiple of 8 channels, at most 8192: a thread owns 8
+// neighbouring channels of both rows in registers.
+__global__ void __launch_bounds__(1024)
+normed_pair_bf16_vec_kernel(const bf16* __restrict__ a, const bf16* __restrict__ b, const float* __restrict__ wa,
+                            const float* __restrict__ wb, float eps, float factor, float* __restrict__ residual,
+                            bf16* __restrict__ out, int H) {
+    chain_release();
+    chain_wait();
+    __shared__ float part[2][32];
+    const int c = threadIdx.x * 8, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const bool active = c < H;
+    const size_t base = (size_t)blockIdx.x * H + c;
+    float x[8], y[8], r[8];
+    float sa = 0.f, sb = 0.f;
+    if (active) {
+        const uint4 ua = *reinterpret_cast<const uint4*>(a + base), ub = *reinterpret_cast<const uint4*>(b + base);
+        if (residual) {
+            const float4 r0 = reinterpret_cast<const float4*>(residual + base)[0], r1 = reinterpret_cast<const float4*>(residual + base)[1];
+            r[0] = r0.x; r[1] = r0.y; r[2] = r0.z; r[3] = r0.w; r[4] = r1.x; r[5] = r1.y; r[6] = r1.z; r[7] = r1.w;
+        }
+        const __nv_bfloat162* ha = reinterpret_cast<const __nv_bfloat162*>(&ua);
+        const __nv_bfloat162* hb = reinterpret_cast<const __nv_bfloat162*>(&ub);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 f = __bfloat1622float2(ha[j]), g = __bfloat1622float2(hb[j]);
+            x[2 * j] = f.x; x[2 * j + 1] = f.y;
+            y[2 * j] = g.x; y[2 * j + 1] = g.y;
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { sa += x[j] * x[j]; sb += y[j] * y[j]; }
+    }
+    sa = warp_sum(sa);
+    sb = warp_sum(sb);
+    if (lane == 0) { part[0][warp] = sa; part[1][warp] = sb; }
+    __syncthreads();
+    if (!active) return;
+    sa = sb = 0.f;
+    for (int w = 0; w < warps; ++w) { sa += part[0][w]; sb += part[1][w]; }
+    sa = factor / sqrtf(sa / (float)H + eps);
+    sb = factor / sqrtf(sb / (float)H + eps);
+    const float4 a0 = reinterpret_cast<const float4*>(wa + c)[0], a1 = reinterpret_cast<const float4*>(wa + c)[1];
+    const float4 b0 = reinterpret_cast<const float4*>(wb + c)[0], b1 = reinterpret_cast<const float4*>(wb + c)[1];
+    const float ua[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+    const float ub[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = x[j] * sa * ua[j] + y[j] * sb * ub[j];
+    if (residual) {
+        reinterpret_cast<float4*>(residual + base)[0] = make_float4(r[0] + v[0], r[1] + v[1], r[2] + v[2], r[3] + v[3]);
+        reinterpret_cast<float4*>(residual + base)[1] = make_float4(r[4] + v[4], r[5] + v[5], r[6] + v[6], r[7] + v[7]);
+    } else {
+        uint4 o;
+        __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) oh[j] = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+        *reinterpret_cast<uint4*>(out + base) = o;
+    }
+}
+
+GTG_API int gtg_normed_pair(int dtype, const void* a, const void* b, const float* wa, const float* wb, float eps, float factor,
+                            float* residual, void* out, int N, int H, cudaStream_t stream) {
+    if (N <= 0) return 0;
+    if (H <= 0 || (residual == nullptr) == (out == nullptr)) return kErrBadArgument;
+    if (dtype == 1 && H % 8 == 0 && H <= 8192 && ((uintptr_t)a % 16) == 0 && ((uintptr_t)b % 16) == 0 && ((uintptr_t)wa % 16) == 0 &&
+        ((uintptr_t)wb % 16) == 0 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)out % 16) == 0)
+        return launch_chained(normed_pair_bf16_vec_kernel, dim3(N), dim3((H / 8 + 31) / 32 * 32), 0, stream, (const bf16*)a, (const bf16*)b,
+                              wa, wb, eps, factor, residual, (bf16*)out, H);
+    int threads = 32;
+    while (threads < 1024 && threads * 4 < H) threads *= 2;
+    const size_t smem = (size_t)(2 * H + 33) * sizeof(float);
+    if (smem > 200 * 1024) return kErrUnsupported;
+#define GTG_PAIR(T)                                                                                                  \
+    do {                                                                                                             \
+        if (smem > 48 * 1024) {                                                                                      \
+            const cudaError_t e = cudaFuncSetAttribute(normed_pair_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                     \
+        }                                                                                                            \
+        return launch_chained(normed_pair_kernel<T>, dim3(N), dim3(threads), smem, stream, (const T*)a, (const T*)b, wa, wb, eps, factor, \
+                              residual, (T*)out, H);                                                                 \
+    } while (0)
+    if (dtype == 0) GTG_PAIR(float);
+    if (dtype == 1) GTG_PAIR(bf16);
+#undef GTG_PAIR
+    return kErrBadArgument;
 }

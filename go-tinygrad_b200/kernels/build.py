@@ -47,6 +47,8 @@ LIBRARIES: Dict[str, str] = {
     "attention_prep": "attention_prep.cu",
     "attention_masked": "attention_masked.cu",
     "delta": "delta.cu",
+    "selective": "selective.cu",
+    "mlstm": "mlstm.cu",
 }
 # sources a library's file includes textually (they count for staleness)
 INCLUDED_SOURCES: Dict[str, List[str]] = {"attention_decode_static.cu": ["attention_bf16.cu"]}

@@ -21,9 +21,10 @@ _P, _I, _L, _F, _U, _D = c_void_p, c_int, c_longlong, c_float, c_ulonglong, c_do
 
 # library, symbol -> argument types (the stream is always last)
 _SIGNATURES = {
-    "gtg_embed": ("elementwise", [_I, _P, _P, _P, _I, _I, _I, _F, _P]),
-    "gtg_add_rmsnorm": ("elementwise", [_I, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
-    "gtg_swiglu": ("elementwise", [_I, _P, _P, _I, _I, _I, _P]),
+    "gtg_embed": ("elementwise", [_I, _P, _P, _P, _I, _I, _I, _F, _P, _P, _P]),
+    "gtg_add_rmsnorm": ("elementwise", [_I, _P, _P, _P, _F, _P, _P, _I, _I, _P, _P, _P]),
+    "gtg_normed_pair": ("elementwise", [_I, _P, _P, _P, _P, _F, _F, _P, _P, _I, _I, _P]),
+    "gtg_swiglu": ("elementwise", [_I, _P, _P, _I, _I, _I, _I, _P]),
     "gtg_rmsnorm_rows": ("elementwise", [_P, _P, _F, _I, _I, _P]),
     "gtg_scale": ("elementwise", [_P, _L, _F, _P]),
     "gtg_rope_table": ("elementwise", [_P, _P, _P, _I, _I, _D, _P]),
@@ -57,13 +58,16 @@ _SIGNATURES = {
     "gtg_gemm_bf16_swapab_scratch_floats": ("gemm_bf16_swapab", [_I, _I, _I]),
     "gtg_gemm_bf16_swapab_status": ("gemm_bf16_swapab", []),
     "gtg_attention_simple": ("attention_simple", [_I, _P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P,
-                                                  _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P, _P]),
+                                                  _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _I, _F, _P, _P, _P]),
+    "gtg_qk_rows_finish": ("attention_prep", [_I, _P, _I, _P, _P, _F, _F, _D, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P]),
     "gtg_qkv_conv_finish": ("attention_prep", [_I, _P, _I, _P, _P, _I, _P, _P, _P, _P, _F, _P, _I, _I, _P, _I, _P, _P, _L, _P, _I,
                                                _P, _P, _P, _I, _I, _I, _I, _I, _I, _P]),
     "gtg_delta_prepare": ("delta", [_P, _I, _P, _I, _P, _P, _P, _I, _P, _I, _I, _I, _I, _F, _F, _P]),
     "gtg_delta_scan_supports": ("delta", [_I, _I]),
     "gtg_delta_scan": ("delta", [_P, _I, _P, _I, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _I, _P]),
-    "gtg_head_norm_gate": ("delta", [_I, _P, _I, _P, _I, _P, _F, _P, _I, _I, _I, _I, _P]),
+    "gtg_head_norm_gate": ("delta", [_I, _I, _P, _I, _P, _I, _P, _I, _F, _P, _P, _I, _I, _I, _I, _P]),
+    "gtg_selective_scan": ("selective", [_I, _P, _I, _P, _I, _P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _P, _P, _I, _I, _I, _I, _P]),
+    "gtg_mlstm_scan": ("mlstm", [_I, _P, _P, _P, _I, _P, _I, _P, _F, _F, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P]),
     "gtg_rmsnorm_add": ("elementwise", [_I, _I, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
     "gtg_round_rows": ("elementwise", [_I, _P, _P, _L, _P]),
     "gtg_swiglu_bias": ("elementwise", [_I, _P, _P, _P, _P, _I, _I, _I, _P]),
@@ -90,7 +94,7 @@ _SIGNATURES = {
     "gtg_attention_masked_scratch_floats": ("attention_masked", [_I, _I, _I, _I]),
     "gtg_attention_masked_splits": ("attention_masked", [_I, _I, _I, _I, _I, _I, _I]),
     "gtg_attention_masked_bf16": ("attention_masked", [_P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
-                                                       _F, _I, _I, _P, _I, _P, _F, _I, _P]),
+                                                       _F, _I, _I, _P, _I, _P, _F, _I, _P, _P]),
     "gtg_hyper_norm": ("hyper", [_I, _I, _P, _P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P]),
     "gtg_qkv_finish": ("attention_prep", [_I, _P, _I, _P, _P, _I, _I, _F, _P, _P, _F, _P, _I, _P, _P, _P, _L, _P, _I, _P, _P, _P,
                                           _I, _I, _I, _I, _I, _P]),
@@ -109,7 +113,7 @@ _SIGNATURES = {
     "gtg_attention_tcgen05_supports": ("attention_tcgen05", [_I]),
     "gtg_attention_tcgen05_status": ("attention_tcgen05", []),
     "gtg_attention_prefill_tcgen05": ("attention_tcgen05", [_P, _I, _I, _P, _I, _P, _P, _L, _I, _P, _I, _P, _P, _P,
-                                                            _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _P]),
+                                                            _I, _I, _I, _I, _I, _F, _I, _I, _P, _F, _I, _P, _P]),
     "gtg_argmax": ("sampling", [_P, _I, _I, _I, _P, _P]),
     "gtg_sample_temperature": ("sampling", [_P, _I, _I, _I, _F, _U, _P, _P, _P, _P]),
 }
@@ -277,19 +281,28 @@ def _check_access(what: str, mode: int, kv, slots, positions=None, token_seq=Non
 
 
 # ------------------------------------------------------------------ elementwise
-def embed(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out[n,:] (float32) = table[tokens[n],:] * scale."""
+def embed(tokens: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float = 1.0,
+          positions: Optional[torch.Tensor] = None, turns: Optional[torch.Tensor] = None) -> None:
+    """out[n,:] (float32) = table[tokens[n],:] * scale; with `turns` (float64 [ceil(H/2)], whole
+    turns a position) channel 2i gets sin(2 pi positions[n] turns[i]) added, channel 2i+1 the cosine."""
     N, (V, H) = tokens.numel(), table.shape
     _need(tokens.dtype == torch.int32 and tokens.is_contiguous(), "embed: tokens must be contiguous int32")
     _need(table.is_contiguous() and out.is_contiguous() and out.dtype == torch.float32
           and tuple(out.shape) == (N, H), "embed: out must be contiguous float32 [N, H]")
-    _check(_fn("gtg_embed")(_dt(table), _ptr(tokens), _ptr(table), _ptr(out), N, H, V, float(scale), _stream()), "embed")
+    if turns is not None:
+        _need(turns.dtype == torch.float64 and turns.is_contiguous() and turns.numel() == (H + 1) // 2, "embed: turns must be float64 [ceil(H/2)]")
+        _need(positions is not None and positions.dtype == torch.int32 and positions.is_contiguous() and positions.numel() == N,
+              "embed: positions must be contiguous int32 [N]")
+    _check(_fn("gtg_embed")(_dt(table), _ptr(tokens), _ptr(table), _ptr(out), N, H, V, float(scale), _ptr(positions), _ptr(turns),
+                            _stream()), "embed")
 
 
 def add_rmsnorm(residual: torch.Tensor, pending: Optional[torch.Tensor], weight: torch.Tensor,
-                eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+                eps: float, out: torch.Tensor, rows: Optional[torch.Tensor] = None,
+                second: Optional[torch.Tensor] = None, out_second: Optional[torch.Tensor] = None) -> None:
     """residual (+= pending); out = rmsnorm(residual) * weight.  With `rows` only
-    those rows are read (nothing is written back) and out has len(rows) rows."""
+    those rows are read (nothing is written back) and out has len(rows) rows.
+    `second`, `out_second`: another weight over the same normed rows and its output."""
     H = residual.shape[1]
     R = rows.numel() if rows is not None else residual.shape[0]
     _need(residual.dtype == torch.float32 and residual.is_contiguous(), "add_rmsnorm: residual must be contiguous float32")
@@ -301,18 +314,40 @@ def add_rmsnorm(residual: torch.Tensor, pending: Optional[torch.Tensor], weight:
               "add_rmsnorm: pending must match the residual's shape and out's dtype")
     if rows is not None:
         _need(rows.dtype == torch.int32 and rows.is_contiguous(), "add_rmsnorm: rows must be contiguous int32")
+    if second is not None:
+        _need(second.dtype == torch.float32 and second.is_contiguous() and second.numel() == H, "add_rmsnorm: the second weight must be float32 [H]")
+        _need(out_second is not None and out_second.is_contiguous() and out_second.shape == out.shape and out_second.dtype == out.dtype,
+              "add_rmsnorm: the second output must match the first")
     _check(_fn("gtg_add_rmsnorm")(_dt(out), _ptr(residual), _ptr(pending), _ptr(weight), float(eps),
-                                  _ptr(out), _ptr(rows), R, H, _stream()), "add_rmsnorm")
+                                  _ptr(out), _ptr(rows), R, H, _ptr(second), _ptr(out_second), _stream()), "add_rmsnorm")
+
+
+def normed_pair(a: torch.Tensor, b: torch.Tensor, weight_a: torch.Tensor, weight_b: torch.Tensor, eps: float, factor: float,
+                residual: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None) -> None:
+    """factor * (rmsnorm(a) * weight_a + rmsnorm(b) * weight_b), in float, added to the float32 rows
+    `residual` or, where that is None, left in `out` (a's dtype)."""
+    N, H = a.shape
+    _need(a.is_contiguous() and b.is_contiguous() and b.shape == a.shape and b.dtype == a.dtype, "normed_pair: a and b must be contiguous and alike")
+    for w in (weight_a, weight_b):
+        _need(w.dtype == torch.float32 and w.is_contiguous() and w.numel() == H, "normed_pair: weights must be float32 [H]")
+    _need((residual is None) != (out is None), "normed_pair: either the residual or an output")
+    if residual is not None:
+        _need(residual.dtype == torch.float32 and residual.is_contiguous() and residual.shape == a.shape, "normed_pair: residual must be contiguous float32")
+    else:
+        _need(out.is_contiguous() and out.shape == a.shape and out.dtype == a.dtype, "normed_pair: out must match a")
+    _check(_fn("gtg_normed_pair")(_dt(a), _ptr(a), _ptr(b), _ptr(weight_a), _ptr(weight_b), float(eps), float(factor), _ptr(residual),
+                                  _ptr(out), N, H, _stream()), "normed_pair")
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
     """out[m,i] = act(gate_up[m,i]) * gate_up[m,I+i], act = silu or another of `ACTIVATIONS`."""
     _need(activation in ACTIVATIONS, f"swiglu: activation {activation!r} is not known; known: {sorted(ACTIVATIONS)}")
     M, two_i = gate_up.shape
-    _need(two_i % 2 == 0 and gate_up.is_contiguous() and out.is_contiguous()
+    _rows2d(out, "swiglu: out")
+    _need(two_i % 2 == 0 and gate_up.is_contiguous()
           and tuple(out.shape) == (M, two_i // 2) and out.dtype == gate_up.dtype,
-          "swiglu: gate_up [M, 2I] and out [M, I] must be contiguous and of one dtype")
-    _check(_fn("gtg_swiglu")(_dt(out), _ptr(gate_up), _ptr(out), M, two_i // 2, ACTIVATIONS[activation], _stream()), "swiglu")
+          "swiglu: gate_up [M, 2I] must be contiguous and out [M, I] of its dtype")
+    _check(_fn("gtg_swiglu")(_dt(out), _ptr(gate_up), _ptr(out), out.stride(0), M, two_i // 2, ACTIVATIONS[activation], _stream()), "swiglu")
 
 
 def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor, amplitude: float = 1.0) -> None:
@@ -641,6 +676,28 @@ def qkv_conv_finish(sums: torch.Tensor, bias: Optional[torch.Tensor], conv_w: Op
 
 
 # ------------------------------------------------------------- the gated delta rule
+def qk_rows_finish(qk: torch.Tensor, q_norm: torch.Tensor, k_norm: torch.Tensor, eps: float, n_heads: int, kv, q_out: torch.Tensor,
+                   token_seq, slots, positions, temperature=None) -> None:
+    """From projected rows [N, q | k]: the queries, RMS-normed over all heads at once with a weight, times
+    1 + coef ln(floor((position + 1) / every) + 1) where `temperature` is (coef, every), to `q_out`; the
+    keys as projected to the value plane of the cache `kv`, normed over all heads at once to its key plane."""
+    _rows2d(qk, "qk_rows_finish: qk"); _rows2d(q_out, "qk_rows_finish: q_out")
+    N = qk.shape[0]
+    hd, n_kv = kv.head_dim, kv.n_kv_heads
+    _need(kv.value_dim == hd, "qk_rows_finish: the values are the keys, so their widths must agree")
+    _need(qk.shape[1] >= (n_heads + n_kv) * hd and q_out.shape[0] == N and q_out.shape[1] >= n_heads * hd, "qk_rows_finish: qk or q_out is too narrow")
+    _need(qk.dtype == q_out.dtype == kv.k.dtype, "qk_rows_finish: one dtype for rows, queries and cache")
+    for w, size in ((q_norm, n_heads * hd), (k_norm, n_kv * hd)):
+        _need(w.dtype == torch.float32 and w.is_contiguous() and w.numel() == size, "qk_rows_finish: norm weights must be float32 of a whole row")
+    coef, every = temperature if temperature else (0.0, 0.0)
+    _int32("qk_rows_finish", token_seq, slots, positions)
+    _check_access("qk_rows_finish", 0, kv, slots, positions, token_seq, n_items=N)
+    _check(_fn("gtg_qk_rows_finish")(_dt(qk), _ptr(qk), qk.stride(0), _ptr(q_norm), _ptr(k_norm), float(eps), float(coef), float(every),
+                                     _ptr(q_out), q_out.stride(0), _ptr(kv.k), _ptr(kv.v), kv.page_stride, _ptr(kv.block_table),
+                                     kv.table_stride, _ptr(token_seq), _ptr(slots), _ptr(positions), N, n_heads, n_kv, hd, _stream()),
+           "qk_rows_finish")
+
+
 DELTA_MAX_KEY_DIM = 512       # most key channels a head of the delta rule's state may have (16 rows a lane, 32 lanes)
 
 
@@ -698,19 +755,83 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, beta: tor
 
 
 def head_norm_gate(y: torch.Tensor, gate_logits: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
-                   n_heads: int) -> None:
+                   n_heads: int, den: Optional[torch.Tensor] = None) -> None:
     """out[n, h, :] = y[n, h, :] / sqrt(mean(y[n, h, :]^2) + eps) * weight * sigmoid(gate_logits[n, h, :]):
-    y and gate_logits float32 [N, heads * dv], weight float32 [dv] shared by the heads."""
+    y float32 [N, heads * dv], gate_logits float32 or out's dtype, weight float32 [dv] shared by the
+    heads or [heads * dv].  With `den` (float32 [N, heads]) a head is divided by its number first."""
     _rows2d(y, "head_norm_gate: y"); _rows2d(gate_logits, "head_norm_gate: gate"); _rows2d(out, "head_norm_gate: out")
     N, width = y.shape
     _need(width % n_heads == 0, "head_norm_gate: the row is not a whole number of heads")
     dv = width // n_heads
-    _need(y.dtype == torch.float32 and gate_logits.dtype == torch.float32 and tuple(gate_logits.shape) == (N, width)
-          and tuple(out.shape) == (N, width), "head_norm_gate: y and gate float32 [N, heads * dv], out of that shape")
-    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == dv,
-          "head_norm_gate: weight must be float32 [dv]")
-    _check(_fn("gtg_head_norm_gate")(_dt(out), _ptr(y), y.stride(0), _ptr(gate_logits), gate_logits.stride(0), _ptr(weight),
-                                     float(eps), _ptr(out), out.stride(0), N, n_heads, dv, _stream()), "head_norm_gate")
+    _need(y.dtype == torch.float32 and gate_logits.dtype in (torch.float32, out.dtype) and tuple(gate_logits.shape) == (N, width)
+          and tuple(out.shape) == (N, width), "head_norm_gate: y float32 [N, heads * dv], gate and out of that shape")
+    _need(weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() in (dv, width),
+          "head_norm_gate: weight must be float32 [dv] or [heads * dv]")
+    _need(den is None or (den.dtype == torch.float32 and den.is_contiguous() and tuple(den.shape) == (N, n_heads)),
+          "head_norm_gate: den must be contiguous float32 [N, heads]")
+    _check(_fn("gtg_head_norm_gate")(_dt(out), 1 if gate_logits.dtype == torch.float32 else 0, _ptr(y), y.stride(0), _ptr(gate_logits),
+                                     gate_logits.stride(0), _ptr(weight), dv if weight.numel() == width else 0, float(eps), _ptr(den),
+                                     _ptr(out), out.stride(0), N, n_heads, dv, _stream()), "head_norm_gate")
+
+
+MLSTM_MAX_KEY_DIM = 512       # most key channels a head of the matrix memory may have (16 rows a lane)
+SELECTIVE_MAX_STATES = 512    # most states a channel of the selective scan may have (16 a lane, 32 lanes)
+
+
+def selective_scan(x: torch.Tensor, bc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, rates: torch.Tensor,
+                   skip: torch.Tensor, z: torch.Tensor, state: torch.Tensor, out: torch.Tensor, cu_seqlens, slots, n_seqs: int,
+                   one_token_each: bool = False) -> None:
+    """The selective scan with its gate: per channel c and state n, dt = softplus(dt_raw + dt_bias),
+    S <- exp(dt rates) S + dt x B, out = (sum_n S C + skip x) silu(z).  x, z, out [n, channels] and
+    bc [n, B | C] of one dtype; dt_raw float32 [n, channels]; rates float32 [channels, N], negative;
+    state float32 [slots, channels, N].  `one_token_each`: row b is sequence b's only token."""
+    for name, t in (("x", x), ("bc", bc), ("dt", dt_raw), ("z", z), ("out", out)):
+        _rows2d(t, f"selective_scan: {name}")
+    n, C = x.shape
+    N = rates.shape[1]
+    _need(x.dtype == bc.dtype == z.dtype == out.dtype and tuple(z.shape) == (n, C) and tuple(out.shape) == (n, C)
+          and tuple(bc.shape) == (n, 2 * N), "selective_scan: x, z, out [n, channels] and bc [n, 2 N] of one dtype")
+    _need(dt_raw.dtype == torch.float32 and tuple(dt_raw.shape) == (n, C), "selective_scan: dt_raw must be float32 [n, channels]")
+    for t, size in ((dt_bias, C), (skip, C), (rates, C * N)):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and t.numel() == size, "selective_scan: bias, skip and rates must be contiguous float32")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (C, N),
+          "selective_scan: state must be float32 [slots, channels, N]")
+    _int32("selective_scan", cu_seqlens, slots)
+    if one_token_each:
+        _need(n == n_seqs, "selective_scan: one token each means as many rows as sequences")
+    _check(_fn("gtg_selective_scan")(_dt(x), _ptr(x), x.stride(0), _ptr(bc), bc.stride(0), _ptr(dt_raw), dt_raw.stride(0), _ptr(dt_bias),
+                                     _ptr(rates), _ptr(skip), _ptr(z), z.stride(0), _ptr(state), _ptr(out), out.stride(0),
+                                     _ptr(cu_seqlens), _ptr(slots), int(n_seqs), C, N, 1 if one_token_each else 0, _stream()),
+           "selective_scan")
+
+
+def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: float,
+               q_scale: float, state, num: torch.Tensor, den: torch.Tensor, cu_seqlens, slots, n_seqs: int, heads: int,
+               one_token_each: bool = False) -> None:
+    """The matrix memory (csrc/mlstm.cu): q, k [n, heads * d] and v [n, heads * dv], columns of one
+    matrix; gates float32 [n, i | f] (heads each, before bias and cap), gate_bias float32 [2 heads];
+    state: (S [slots, heads, d, dv], n [slots, heads, d], m [slots, heads, dv + 1]), float32.  Leaves
+    num = S^T q float32 [n, heads * dv] and den float32 [n, heads], the quotient's other half."""
+    for name, t in (("q", q), ("k", k), ("v", v), ("gates", gates), ("num", num)):
+        _rows2d(t, f"mlstm_scan: {name}")
+    n = q.shape[0]
+    _need(q.shape[1] % heads == 0 and v.shape[1] % heads == 0 and k.shape == q.shape and v.shape[0] == n, "mlstm_scan: q, k and v do not fit the heads")
+    d, dv = q.shape[1] // heads, v.shape[1] // heads
+    _need(q.dtype == k.dtype == v.dtype and q.stride(0) == k.stride(0) == v.stride(0), "mlstm_scan: q, k and v must be columns of one matrix")
+    _need(gates.dtype == torch.float32 and tuple(gates.shape) == (n, 2 * heads), "mlstm_scan: gates must be float32 [n, 2 heads]")
+    _need(gate_bias.dtype == torch.float32 and gate_bias.is_contiguous() and gate_bias.numel() == 2 * heads, "mlstm_scan: gate_bias must be float32 [2 heads]")
+    _need(num.dtype == torch.float32 and tuple(num.shape) == (n, heads * dv), "mlstm_scan: num must be float32 [n, heads * dv]")
+    _need(den.dtype == torch.float32 and den.is_contiguous() and tuple(den.shape) == (n, heads), "mlstm_scan: den must be contiguous float32 [n, heads]")
+    S, nn, m = state
+    for t, shape in ((S, (heads, d, dv)), (nn, (heads, d)), (m, (heads, dv + 1))):
+        _need(t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape[1:]) == shape, f"mlstm_scan: a state must be float32 [slots, {shape}]")
+    _need(d <= MLSTM_MAX_KEY_DIM, f"mlstm_scan: heads of {d} key channels exceed {MLSTM_MAX_KEY_DIM}")
+    _int32("mlstm_scan", cu_seqlens, slots)
+    if one_token_each:
+        _need(n == n_seqs, "mlstm_scan: one token each means as many rows as sequences")
+    _check(_fn("gtg_mlstm_scan")(_dt(q), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(gates), gates.stride(0), _ptr(gate_bias), float(cap),
+                                 float(q_scale), _ptr(S), _ptr(nn), _ptr(m), _ptr(num), num.stride(0), _ptr(den), _ptr(cu_seqlens),
+                                 _ptr(slots), int(n_seqs), heads, d, dv, 1 if one_token_each else 0, _stream()), "mlstm_scan")
 
 
 # ------------------------------------------------------------- recurrent mixers
@@ -1045,10 +1166,16 @@ def attention_bf16_supports(head_dim: int) -> bool:
     return bool(_fn("gtg_attention_bf16_supports")(head_dim))
 
 
+def _need_slopes(slopes: Optional[torch.Tensor], n_heads: int) -> None:
+    _need(slopes is None or (slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == n_heads),
+          "attention: slopes must be contiguous float32 [n_heads]")
+
+
 def attention_simple(q: torch.Tensor, out: torch.Tensor, kv, token_seq, slots, positions,
                      n_heads: int, scale: float, window: int = 0, value_dim: Optional[int] = None,
                      chunk: int = 0, gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                     sinks: Optional[torch.Tensor] = None, gate_logits: Optional[torch.Tensor] = None) -> None:
+                     sinks: Optional[torch.Tensor] = None, gate_logits: Optional[torch.Tensor] = None,
+                     slopes: Optional[torch.Tensor] = None) -> None:
     """One warp per (token, head): the float32 path's attention, for prompts and
     decode steps alike.  `value_dim`: a value is the first so many channels of a
     row of the value plane (default: all of them), and a head of `out` is that wide.
@@ -1056,8 +1183,10 @@ def attention_simple(q: torch.Tensor, out: torch.Tensor, kv, token_seq, slots, p
     `gate`: float32 [N, n_heads], a factor on each head's output; `gate_logits`: float32
     rows of n_heads * value width logits (any row stride) whose sigmoids multiply the
     output channel by channel.  `softcap` c > 0: scores become c tanh(score / c).
-    `sinks`: float32 [n_heads]; exp(sinks[h]) joins head h's softmax denominator."""
+    `sinks`: float32 [n_heads]; exp(sinks[h]) joins head h's softmax denominator.  `slopes`: float32
+    [n_heads]; slopes[h] times the distance between query and key is taken off the score."""
     _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
+    _need_slopes(slopes, n_heads)
     N = q.shape[0]
     vrow = kv.value_dim
     vd = vrow if value_dim is None else int(value_dim)
@@ -1082,13 +1211,13 @@ def attention_simple(q: torch.Tensor, out: torch.Tensor, kv, token_seq, slots, p
                                        _ptr(kv.k), _ptr(kv.v), kv.page_stride, _ptr(kv.block_table),
                                        kv.table_stride, _ptr(token_seq), _ptr(slots), _ptr(positions),
                                        N, n_heads, kv.n_kv_heads, kv.head_dim, vd, vrow, float(scale), int(window),
-                                       int(chunk), _ptr(gate), int(gate_ld), float(softcap), _ptr(sinks), _stream()),
+                                       int(chunk), _ptr(gate), int(gate_ld), float(softcap), _ptr(sinks), _ptr(slopes), _stream()),
            "attention_simple")
 
 
 def attention_general(q: torch.Tensor, out: torch.Tensor, kv, ctx, n_heads: int, scale: float, window: int = 0,
                       chunk: int = 0, gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                      gate_logits: Optional[torch.Tensor] = None) -> None:
+                      gate_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> None:
     """Attention for mixers whose keys and values differ in size, whose keys are seen
     within stretches of `chunk` positions, or whose heads carry a gate: `ctx` is the
     step's context (rows, positions, sequences).  out[n, h] = gate[n, h] *
@@ -1097,14 +1226,15 @@ def attention_general(q: torch.Tensor, out: torch.Tensor, kv, ctx, n_heads: int,
     and other widths the plain one; steps that bring more than one token a sequence, with
     keys and values of 64 or 128 channels alike, the prompt attention on tcgen05.
     `softcap` c > 0: scores become c tanh(score / c) after the scale.  `gate_logits`: float32
-    rows [N, n_heads * value width] whose sigmoids multiply the output channel by channel."""
+    rows [N, n_heads * value width] whose sigmoids multiply the output channel by channel.
+    `slopes`: float32 [n_heads], a penalty on the distance of query and key per head."""
     if (q.dtype == torch.bfloat16 and not ctx.is_decode and kv.value_dim == kv.head_dim and attention_tcgen05_supports(kv)
             and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
         # the logits' sigmoids multiply the output in a kernel of their own here: in this kernel's epilogue a thread
         # holds a query's row and reads its 64 or 128 logits alone, which cost the kernel 37 us of 94 at 2,048 tokens
         # against 10 us for the pass over rows
         attention_prefill_tcgen05(q, out, kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, ctx.n_seqs, ctx.max_q_len, n_heads, scale,
-                                  window, chunk, gate, softcap=softcap)
+                                  window, chunk, gate, softcap=softcap, slopes=slopes)
         if gate_logits is not None:
             sigmoid_gate(out[:, : n_heads * kv.value_dim], gate_logits)
         return
@@ -1116,10 +1246,10 @@ def attention_general(q: torch.Tensor, out: torch.Tensor, kv, ctx, n_heads: int,
             scratch = ctx.rt.empty(int(_fn("gtg_attention_masked_scratch_floats")(q.shape[0], n_heads, kv.value_dim, splits)),
                                    dtype=torch.float32)
         attention_masked_bf16(q, out, kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, ctx.n_seqs, ctx.max_q_len, n_heads, scale,
-                              window, chunk, gate, splits, scratch, softcap=softcap, gate_logits=gate_logits)
+                              window, chunk, gate, splits, scratch, softcap=softcap, gate_logits=gate_logits, slopes=slopes)
         return
     attention_simple(q, out, kv, ctx.token_seq, ctx.slots, ctx.positions, n_heads, scale, window, chunk=chunk, gate=gate,
-                     softcap=softcap, gate_logits=gate_logits)
+                     softcap=softcap, gate_logits=gate_logits, slopes=slopes)
 
 
 def attention_masked_supports(kv) -> bool:
@@ -1130,12 +1260,13 @@ def attention_masked_supports(kv) -> bool:
 def attention_masked_bf16(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: int, max_q_len: int, n_heads: int, scale: float,
                           window: int = 0, chunk: int = 0, gate: Optional[torch.Tensor] = None, n_splits: int = 1,
                           scratch: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                          gate_logits: Optional[torch.Tensor] = None) -> None:
+                          gate_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> None:
     """The tensor-core form of `attention_general`: rows are (token, query head of a group)
     pairs, a block of 64 rows reads each page once for the group.  Prompts, portions and
     decode steps alike; `n_splits` > 1 cuts every tile's pages into that many shares, merged
-    through `scratch` (float32, `gtg_attention_masked_scratch_floats`).  `softcap` and
-    `gate_logits` as in `attention_simple`."""
+    through `scratch` (float32, `gtg_attention_masked_scratch_floats`).  `softcap`, `gate_logits`
+    and `slopes` as in `attention_simple`."""
+    _need_slopes(slopes, n_heads)
     _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
     N = q.shape[0]
     gate_ld = 0
@@ -1161,7 +1292,7 @@ def attention_masked_bf16(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: int,
                                             _ptr(kv.block_table), kv.table_stride, _ptr(cu_seqlens), _ptr(slots), _ptr(start_pos),
                                             int(n_seqs), int(max_q_len), N, n_heads, kv.n_kv_heads, kv.head_dim, kv.value_dim,
                                             float(scale), int(window), int(chunk), _ptr(gate), int(n_splits), _ptr(scratch),
-                                            float(softcap), int(gate_ld), _stream()),
+                                            float(softcap), int(gate_ld), _ptr(slopes), _stream()),
            "attention_masked_bf16")
 
 
@@ -1192,11 +1323,12 @@ def attention_tcgen05_supports(kv) -> bool:
 def attention_prefill_tcgen05(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: int, max_q_len: int,
                               n_heads: int, scale: float, window: int = 0, chunk: int = 0,
                               gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                              gate_logits: Optional[torch.Tensor] = None) -> None:
+                              gate_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None) -> None:
     """Prompt attention on tcgen05 (128 queries x one head per thread block).  `chunk` > 0:
     a query sees the keys of its own stretch of `chunk` positions only; `gate`: float32
-    [N, n_heads], a factor on each head's output.  `softcap` and `gate_logits` as in
+    [N, n_heads], a factor on each head's output.  `softcap`, `gate_logits` and `slopes` as in
     `attention_simple`."""
+    _need_slopes(slopes, n_heads)
     _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
     gate_ld = 0
     if gate_logits is not None:
@@ -1217,7 +1349,7 @@ def attention_prefill_tcgen05(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: 
                                                 _ptr(kv.block_table), kv.table_stride, _ptr(cu_seqlens),
                                                 _ptr(slots), _ptr(start_pos), n_seqs, max_q_len, n_heads,
                                                 kv.n_kv_heads, kv.head_dim, float(scale), int(window), int(chunk),
-                                                _ptr(gate), float(softcap), int(gate_ld), _stream()),
+                                                _ptr(gate), float(softcap), int(gate_ld), _ptr(slopes), _stream()),
            "attention_prefill_tcgen05")
 
 

@@ -54,6 +54,16 @@ queries, convolution state, window and gate of its own.  ``cache_window`` (where
 given): how many keys the cache keeps for this layer's storage instead of
 ``window`` (None: all of them): a layer whose keys other layers read through
 longer windows, or through none, must keep what the longest-sighted of them sees.
+
+A third family (`_forward_rows`; `ops.qk_rows_finish` stands between projection and
+attention): ``qk_norm`` "rows" with ``q_norm`` and ``k_norm`` (tensor names, as wide
+as all query or all key heads): an RMS norm over the whole row of q and of k before
+it is cut into heads, eps ``norm_eps``; values from the keys, as projected and
+before the norm; no rotation.  With it go ``q_temperature`` (coef, every): queries
+times 1 + coef ln(floor((p + 1) / every) + 1) at position p; and ``distance_slopes``:
+True takes 2^(-8 (h + 1) / n_heads) times the distance between query and key off the
+scores of head h.  A mixer of this family can be handed its projected rows by a part
+that projects for several (`input_matrix`, `forward_projected`).
 """
 from __future__ import annotations
 
@@ -104,8 +114,8 @@ class GQAttention(Mixer):
             raise ValueError("an attention mixer has biases on q, k and v or on none of them")
         self.bias_names = [str(b) for b in biases] if all(biases) else None
         self.qk_norm = self.p.get("qk_norm")
-        if self.qk_norm not in (None, "unit", "weight"):
-            raise ValueError(f"qk_norm {self.qk_norm!r} is not known: None, 'unit' or 'weight'")
+        if self.qk_norm not in (None, "unit", "weight", "rows"):
+            raise ValueError(f"qk_norm {self.qk_norm!r} is not known: None, 'unit', 'weight' or 'rows'")
         conv = self.p.get("conv")
         self.conv = dict(conv) if conv and int(conv.get("taps", 0)) > 0 else None
         self.taps = int(self.conv["taps"]) if self.conv else 1
@@ -124,7 +134,19 @@ class GQAttention(Mixer):
         self.blend = dict(blend) if blend else None
         if self.blend and self.blend.get("role") not in ("source", "blend"):
             raise ValueError(f"value_blend role {self.blend.get('role')!r} is not known: 'source' or 'blend'")
-        self.general = bool(self.value_dim != self.head_dim or self.bias_names or self.qk_norm or self.chunk
+        self.rows_route = self.qk_norm == "rows"
+        temperature = self.p.get("q_temperature")
+        self.temperature = (float(temperature[0]), float(temperature[1])) if temperature else None
+        self.sloped = bool(self.p.get("distance_slopes", False))
+        self.slopes: Optional[torch.Tensor] = None
+        self.shares_input = False             # True once another part projects for this one
+        if (self.temperature or self.sloped) and not self.rows_route:
+            raise ValueError("a query temperature and a penalty on the distance are built with norms over whole rows only")
+        if self.rows_route and (self.conv_route or self.bias_names or self.chunk or self.gate_name or self.blend or not self.v_from_k
+                                or not self.own_kv or self.value_dim != self.head_dim or self.position.kind != "none"):
+            raise ValueError("norms over whole rows of queries and keys are built for unrotated keys that are the values too, without "
+                             "the other options")
+        self.general = not self.rows_route and bool(self.value_dim != self.head_dim or self.bias_names or self.qk_norm or self.chunk
                             or self.gate_name or self.blend or self.conv_route)
         if self.conv_route and (self.qk_norm == "unit" or self.chunk or self.gate_name or self.blend or self.v_from_k):
             raise ValueError("convolved projections, weighted head norms, capped scores and the gate on all channels are "
@@ -132,7 +154,7 @@ class GQAttention(Mixer):
         if self.general and (self.v_from_k or (not self.own_kv and not self.conv_route)):
             raise ValueError("the options of the general attention route need key and value projections of the layer's own")
         self.norm_names = None
-        if self.qk_norm == "weight":
+        if self.qk_norm in ("weight", "rows"):
             self.norm_names = [str(self.param("q_norm"))] + ([str(self.param("k_norm"))] if self.own_kv else [])
         # channels that pass the convolution: q, and k and v where the layer has them
         self.conv_channels = self.q_dim + ((self.kv_dim + self.v_width) if self.own_kv else 0)
@@ -156,7 +178,8 @@ class GQAttention(Mixer):
             specs += [WeightSpec(str(self.conv[k]), (size, self.taps), role="parameter", mean=1.0 / self.taps, std=0.3)
                       for k, size in self._conv_parts()]
         if self.norm_names:
-            specs += [WeightSpec(name, (self.head_dim,), role="vector", mean=1.0) for name in self.norm_names]
+            sizes = (self.q_dim, self.kv_dim) if self.rows_route else (self.head_dim, self.head_dim)
+            specs += [WeightSpec(name, (size,), role="vector", mean=1.0) for name, size in zip(self.norm_names, sizes)]
         if self.out_gate_name:
             specs.append(WeightSpec(self.out_gate_name, (self.n_heads * self.value_dim, self.hidden)))
         if self.gate_name:
@@ -201,10 +224,13 @@ class GQAttention(Mixer):
         if self.out_gate_name:
             parts.append(tensors[self.out_gate_name])
         rows = sum(p.shape[0] for p in parts)
-        if self.general and rows % 8:
+        if (self.general or self.rows_route) and rows % 8:
             # whole groups of 8 rows, so that the products' float sums keep rows of a multiple of 32 bytes
             parts.append(torch.zeros((8 - rows % 8, self.hidden), dtype=parts[0].dtype, device=parts[0].device))
-        self.w_qkv = rt.matrix(torch.cat([p.to(rt.dtype) for p in parts], dim=0))
+        if not self.shares_input:
+            self.w_qkv = rt.matrix(torch.cat([p.to(rt.dtype) for p in parts], dim=0))
+        if self.sloped:
+            self.slopes = rt.vector(torch.tensor([2.0 ** (-8.0 * (h + 1) / self.n_heads) for h in range(self.n_heads)], dtype=torch.float64))
         self.w_o = rt.matrix(tensors[self.names["o"]])
         if self.bias_names:
             self.bias = rt.vector(torch.cat([tensors[name].reshape(-1).to(torch.float32) for name in self.bias_names]))
@@ -241,6 +267,32 @@ class GQAttention(Mixer):
                               softcap=self.softcap, gate_logits=logits)
         ctx.trace("attn", mixed)
         return emit_update(mixed, self.w_o, ctx)
+
+    def input_matrix(self, tensors: Mapping[str, torch.Tensor]) -> List[torch.Tensor]:
+        """The matrices whose products with x, side by side, `forward_projected` reads; None if it cannot be handed them."""
+        return [tensors[self.names["q"]], tensors[self.names["k"]]]
+
+    @property
+    def input_width(self) -> int:
+        return self.q_dim + self.kv_dim
+
+    def forward_projected(self, qk: torch.Tensor, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        rt, kv, n = ctx.rt, cache.kv, qk.shape[0]
+        if not cache.writes:
+            raise ValueError("a mixer with norms over whole rows keeps keys and values of its own")
+        q = rt.empty(n, (self.q_dim + 7) // 8 * 8)[:, : self.q_dim]
+        ops.qk_rows_finish(qk, self.q_norm_w, self.k_norm_w, self.norm_eps, self.n_heads, kv, q, ctx.token_seq, ctx.slots,
+                           ctx.positions, self.temperature)
+        ctx.trace("q_attn", q)
+        mixed = rt.empty(n, (self.q_dim + 7) // 8 * 8)[:, : self.q_dim]
+        ops.attention_general(q, mixed, kv, ctx, self.n_heads, self.scale, window=self.window or 0, slopes=self.slopes)
+        ctx.trace("attn", mixed)
+        return emit_update(mixed, self.w_o, ctx)
+
+    def _forward_rows(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        qk = ctx.rt.empty(x.shape[0], self.w_qkv.shape[0])
+        ops.linear(x, self.w_qkv, qk)
+        return self.forward_projected(qk[:, : self.input_width], x, ctx, cache)
 
     def _forward_general(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
         rt = ctx.rt
@@ -282,6 +334,8 @@ class GQAttention(Mixer):
         kv = cache.kv
         if kv is None or kv.n_kv_heads != self.n_kv or kv.head_dim != self.head_dim or kv.value_dim != self.value_dim:
             raise ValueError("attention was given a cache entry that does not match its heads")
+        if self.rows_route:
+            return self._forward_rows(x, ctx, cache)
         if self.conv_route:
             return self._forward_conv(x, ctx, cache)
         if self.general:

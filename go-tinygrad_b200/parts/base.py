@@ -207,6 +207,9 @@ class StepContext:
     # with float_updates: a bias (float32 [H]) that the part leaves for the block's norm kernel to add to
     # the update it returns, instead of adding it itself; the block takes it and sets this None again
     update_bias: Optional[torch.Tensor] = None
+    # set by a block that multiplies the operands of its sublayers' last products, side by side, with their
+    # matrices side by side: see JointUpdate, update_operand and emit_update
+    joint: Optional["JointUpdate"] = None
     step: int = 0               # which step of the model this is (counted by the model; for `op_hook`)
     layer: int = -1             # the layer that is running (set by the engine before each block)
     op_hook: Optional[Callable[[int, int, str, torch.Tensor], None]] = None
@@ -232,6 +235,8 @@ class Part:
     # rows by data): a step that contains it cannot be recorded as a CUDA graph,
     # and the generation loop then launches its decode steps kernel by kernel.
     capturable: bool = True
+    # True once a block has taken the matrix of this part's last product into a joint one
+    joined: bool = False
 
     def __init__(self, spec: PartSpec):
         self.spec = spec
@@ -249,6 +254,11 @@ class Part:
 
     def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
         """Take the declared tensors (host, stored dtype) and keep what `forward` needs."""
+
+    def last_product(self) -> Optional[Tuple[str, int]]:
+        """(tensor name, inner size) of the matrix whose product is this part's update, for a part
+        that asks `update_operand` where to leave that product's operand; None for any other."""
+        return None
 
     def param(self, name: str, default: Any = None) -> Any:
         if name in self.p:
@@ -289,12 +299,60 @@ class ResidualStream:
         self.pending_links = None
 
 
-def emit_update(x: torch.Tensor, w: torch.Tensor, ctx: "StepContext") -> Optional[torch.Tensor]:
+class JointUpdate:
+    """The operands of several sublayers' last products side by side in one row, so that one product
+    with their matrices side by side gives the sum of their updates.  Every operand starts at a
+    multiple of 8 channels; the channels between are zero in the row and in the matrix."""
+
+    def __init__(self, rt: "Runtime", n: int, widths: List[int]):
+        self.starts = self.starts_of(widths)
+        self.buffer = rt.empty(n, self.starts[-1])
+        self.widths, self.next = list(widths), 0
+        for start, end, width in zip(self.starts, self.starts[1:], widths):
+            if start + width < end:
+                self.buffer[:, start + width: end].zero_()
+
+    @staticmethod
+    def starts_of(widths: List[int]) -> List[int]:
+        starts = [0]
+        for width in widths:
+            starts.append(starts[-1] + (width + 7) // 8 * 8)
+        return starts
+
+    @staticmethod
+    def matrix(matrices: List[torch.Tensor], rt: "Runtime") -> torch.Tensor:
+        """The matrices [hidden, width] side by side."""
+        starts = JointUpdate.starts_of([m.shape[1] for m in matrices])
+        out = torch.zeros((matrices[0].shape[0], starts[-1]), dtype=rt.dtype, device=matrices[0].device)
+        for m, start in zip(matrices, starts):
+            out[:, start: start + m.shape[1]] = m.to(rt.dtype)
+        return rt.matrix(out)
+
+    def take(self, width: int) -> torch.Tensor:
+        if self.next >= len(self.widths) or self.widths[self.next] != width:
+            raise ValueError(f"no operand of {width} channels is expected here: {self.widths}, {self.next} of them taken")
+        start = self.starts[self.next]
+        self.next += 1
+        return self.buffer[:, start: start + width]
+
+
+def update_operand(ctx: "StepContext", n: int, width: int) -> torch.Tensor:
+    """Where a part leaves the operand of its last product (see `Part.last_product`)."""
+    if ctx.joint is not None:
+        return ctx.joint.take(width)
+    return ctx.rt.empty(n, (width + 7) // 8 * 8)[:, :width]
+
+
+def emit_update(x: torch.Tensor, w: Optional[torch.Tensor], ctx: "StepContext") -> Optional[torch.Tensor]:
     """The last product of a mixer or feed-forward: its update x . w^T, [n_tokens, H].
     When the block has offered its residual stream (`ctx.update_into`) and the
     product can add to it in its epilogue (a prompt step in bfloat16), the update
     is added there and None is returned in its place: it never goes through
-    memory, and the norm that follows has nothing left to add."""
+    memory, and the norm that follows has nothing left to add.  Within a joint
+    update (`ctx.joint`) the operand already lies where the block wants it: nothing
+    happens here and None is returned."""
+    if ctx.joint is not None:
+        return None
     stream = ctx.update_into
     if (stream is not None and stream.pending is None and ctx.rt.dtype == torch.bfloat16
             and ops.linear_add_residual(x, w, stream.residual)):
@@ -326,6 +384,9 @@ class PositionEncoding(Part):
     # the whole head; otherwise the first `rotary_dim` channels, the rest pass.
     pairing: str = "half"
     rotary_dim: Optional[int] = None
+    # For absolute encodings that are added to the embedded tokens by the embedding kernel itself:
+    # float64 [ceil(H / 2)] on the device, whole turns a position, channel 2i the sine, 2i + 1 the cosine.
+    embedding_turns: Optional[torch.Tensor] = None
 
     def on_embedding(self, stream: ResidualStream, ctx: StepContext) -> None:
         """Hook for encodings that act on the embedded tokens (absolute positions)."""

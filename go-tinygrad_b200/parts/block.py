@@ -10,6 +10,14 @@ one, or the final one) adds it in float32 while it normalises -- unless the
 part, offered the stream (`emit_update`), has added its update in its last
 product's epilogue already and returns None.
 
+``parallel_pre_norm``: x += mixer(norm1(x)) + feed_forward(norm2(x)), both of the
+same x.  Same four nested specs as ``pre_norm``; the feed-forward and its norm may
+be None.  Both norms come from one pass over the hidden state, and where mixer and
+feed-forward both end in a plain product (`Part.last_product`) one product over
+their operands side by side gives the sum of their updates (`JointUpdate`).  A
+mixer that adds its update to the stream it is offered, or returns one, goes with
+it too.  The reference has no such arrangement.
+
 ``output_norm``: x += norm1(mixer(x)); x += norm2(feed_forward(x)): the norm
 stands on a sublayer's output and the sublayers read the hidden state itself
 (rounded to the compute dtype for their products).  Same four nested specs as
@@ -54,7 +62,7 @@ import torch
 from ..cache import CacheHandle
 from ..kernels import ops
 from ..weights.binder import WeightSpec
-from .base import Block, ResidualStream, Runtime, StepContext, register_part
+from .base import Block, JointUpdate, ResidualStream, Runtime, StepContext, emit_update, register_part
 
 
 def _hidden(stream: ResidualStream):
@@ -85,6 +93,54 @@ class PreNormBlock(Block):
                 stream.pending = self.feed_forward.forward(x, ctx)
                 if stream.pending is not None:
                     ctx.trace("down", stream.pending)
+        finally:
+            ctx.update_into = None
+        ctx.trace("hidden_post_ffn", lambda: _hidden(stream))
+
+
+@register_part("block", "parallel_pre_norm")
+class ParallelPreNormBlock(Block):
+    sub_parts = (("mixer_norm", "norm"), ("mixer", "mixer"),
+                 ("feed_forward_norm", "norm"), ("feed_forward", "feed_forward"))
+    optional_parts = ("feed_forward_norm", "feed_forward")
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.w_joint: Optional[torch.Tensor] = None
+        lasts = [part.last_product() for part in (self.mixer, self.feed_forward) if part is not None]
+        self.lasts = lasts if len(lasts) == 2 and all(lasts) else None
+
+    def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        if self.lasts:                     # before the parts themselves load: they keep no matrix of their own then
+            self.w_joint = JointUpdate.matrix([tensors[name] for name, _ in self.lasts], rt)
+            self.mixer.joined = self.feed_forward.joined = True
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache: CacheHandle) -> None:
+        ctx.trace("hidden_in", lambda: _hidden(stream))
+        if self.feed_forward is not None:
+            x, y = self.mixer_norm.forward_pair(stream, ctx, self.feed_forward_norm)
+            ctx.trace("mlp_input", y)
+        else:
+            x = self.mixer_norm.forward(stream, ctx)
+        ctx.trace("normed", x)
+        if self.w_joint is not None:
+            joint = ctx.joint = JointUpdate(ctx.rt, x.shape[0], [width for _, width in self.lasts])
+            try:
+                self.mixer.forward(x, ctx, cache)
+                self.feed_forward.forward(y, ctx)
+            finally:
+                ctx.joint = None
+        ctx.update_into = stream
+        try:
+            if self.w_joint is not None:
+                stream.pending = emit_update(joint.buffer, self.w_joint, ctx)
+            else:
+                stream.pending = self.mixer.forward(x, ctx, cache)
+                if self.feed_forward is not None:
+                    if stream.pending is not None:          # a mixer that left its update for later: added before the next one
+                        stream.residual += stream.pending.float()
+                        stream.pending, stream.image = None, None
+                    stream.pending = self.feed_forward.forward(y, ctx)
         finally:
             ctx.update_into = None
         ctx.trace("hidden_post_ffn", lambda: _hidden(stream))

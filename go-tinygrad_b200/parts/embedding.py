@@ -4,7 +4,8 @@
 or E[token] * ``scale`` where a scale is given;
 it starts the float32 residual stream.  Parameters: ``vocab_size``,
 ``hidden_size``, ``weight`` and optionally ``scale``, ``position`` (a position PartSpec
-whose `on_embedding` hook acts on the embedded tokens), ``keep_output``
+whose `on_embedding` hook acts on the embedded tokens, or whose `embedding_turns` the
+embedding kernel adds as sinusoids), ``keep_output``
 (True: a float32 copy of the embedded tokens stays in the step's shared values
 as "embedding_output" for later parts to read) and ``norm`` ({"weight": tensor
 name, "eps": e}: the embedded tokens pass an RMS norm with that weight, in
@@ -63,12 +64,13 @@ class TokenEmbedding(Embedding):
 
     def forward(self, ctx: StepContext) -> ResidualStream:
         residual = ctx.rt.empty(ctx.n_tokens, self.hidden, dtype=torch.float32, lifetime="step")
-        ops.embed(ctx.tokens, self.table, residual, self.scale)
+        turns = self.position.embedding_turns if self.position else None
+        ops.embed(ctx.tokens, self.table, residual, self.scale, ctx.positions, turns)
         if self.norm_weight is not None:
             ops.rmsnorm_rows(residual, self.norm_weight, self.norm_eps)
         if self.keep_output:
             kept = ctx.rt.empty(ctx.n_tokens, self.hidden, dtype=torch.float32, lifetime="step")
-            ops.embed(ctx.tokens, self.table, kept, self.scale)
+            ops.embed(ctx.tokens, self.table, kept, self.scale, ctx.positions, turns)
             ctx.shared["embedding_output"] = kept
         stream = ResidualStream(residual)
         if self.position:

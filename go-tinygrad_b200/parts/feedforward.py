@@ -49,7 +49,7 @@ import torch
 
 from ..kernels import ops
 from ..weights.binder import WeightSpec
-from .base import FeedForward, Runtime, StepContext, emit_update, register_part
+from .base import FeedForward, Runtime, StepContext, emit_update, register_part, update_operand
 
 
 @register_part("feed_forward", "swiglu")
@@ -94,14 +94,18 @@ class SwiGLU(FeedForward):
             self.w_gate_up = rt.matrix(ops.interleave_gate_up(gate, up))
         else:
             self.w_gate_up = rt.matrix(torch.cat([gate, up], dim=0))
-        self.w_down = rt.matrix(tensors[self.names["down"]])
+        if not self.joined:
+            self.w_down = rt.matrix(tensors[self.names["down"]])
+
+    def last_product(self):
+        return None if self.bias_names else (self.names["down"], self.inter)
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         rt = ctx.rt
         n = x.shape[0]
         if self.biases:
             return self._forward_biased(x, ctx)
-        act = rt.empty(n, self.inter)
+        act = update_operand(ctx, n, self.inter)
         if self.fused:
             ops.linear(x, self.w_gate_up, act, epilogue=ops.GATED_EPILOGUES[self.activation])
         else:

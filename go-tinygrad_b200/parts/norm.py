@@ -2,7 +2,9 @@
 
 ``rmsnorm``: y = w * x * (1/sqrt(mean(x^2) + eps)) with the sum of squares and
 the scale in float32 (backends/simd/vec.go:72-85).  Parameters: ``size``,
-``eps``, ``weight`` (tensor name).
+``eps``, ``weight`` (tensor name) and optionally ``weight_offset`` (added to the
+stored weight: 1 for a checkpoint that keeps its weights around zero).  Two such
+norms of one hidden state come from one pass (`forward_pair`).
 
 Handed a stream whose hidden state is kept in several copies
 (`ResidualStream.copies`), ``rmsnorm`` norms their sum and applies a pending
@@ -31,13 +33,27 @@ class RMSNorm(Norm):
         self.size = int(self.param("size"))
         self.eps = float(self.param("eps"))
         self.weight_name = str(self.param("weight"))
+        self.offset = float(self.p.get("weight_offset") or 0.0)
         self.weight: Optional[torch.Tensor] = None
 
     def weight_specs(self) -> List[WeightSpec]:
-        return [WeightSpec(self.weight_name, (self.size,), role="vector", mean=1.0)]
+        return [WeightSpec(self.weight_name, (self.size,), role="vector", mean=1.0 - self.offset)]
 
     def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
-        self.weight = rt.vector(tensors[self.weight_name])
+        w = tensors[self.weight_name]
+        self.weight = rt.vector(w.to(torch.float32) + self.offset if self.offset else w)
+
+    def forward_pair(self, stream: ResidualStream, ctx: StepContext, other: "Norm"):
+        """(this norm's rows, `other`'s rows) of the same hidden state, from one pass where both are of this kind."""
+        if not isinstance(other, RMSNorm) or other.eps != self.eps or stream.copies is not None:
+            return self.forward(stream, ctx), other.forward(stream, ctx)
+        n = stream.residual.shape[0]
+        out, out2 = ctx.rt.empty(n, self.size), ctx.rt.empty(n, self.size)
+        ops.add_rmsnorm(stream.residual, stream.pending, self.weight, self.eps, out, second=other.weight, out_second=out2)
+        if stream.pending is not None:
+            stream.image = None
+        stream.pending = None
+        return out, out2
 
     def forward(self, stream: ResidualStream, ctx: StepContext,
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:

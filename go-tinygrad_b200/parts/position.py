@@ -28,6 +28,11 @@ and the frequency is f_i (1 - r_i) + f_i / factor * r_i.  Cosines and sines
 are multiplied by 0.1 ln(factor) + 1, which sharpens the attention as the
 context is stretched.
 
+``sinusoidal``: absolute positions, added to the embedded tokens: channel 2i gets
+sin(p f_i), channel 2i+1 cos(p f_i), f_i = base^(-2i/size).  Queries and keys are
+not rotated.  Parameters: ``size`` (of the hidden state), ``base``.  The embedding
+kernel adds them (`PositionEncoding.embedding_turns`).  Not in the reference.
+
 ``none``: no position encoding.
 """
 from __future__ import annotations
@@ -121,3 +126,15 @@ class RotaryEncoding(PositionEncoding):
 @register_part("position", "none")
 class NoPosition(PositionEncoding):
     pass
+
+
+@register_part("position", "sinusoidal")
+class SinusoidalEncoding(PositionEncoding):
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.size = int(self.param("size"))
+        self.base = float(self.param("base"))
+
+    def load(self, tensors, rt: Runtime) -> None:
+        turns = [math.pow(self.base, -2.0 * i / self.size) / (2.0 * math.pi) for i in range((self.size + 1) // 2)]
+        self.embedding_turns = torch.tensor(turns, dtype=torch.float64, device=rt.device)

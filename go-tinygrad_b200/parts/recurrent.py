@@ -33,7 +33,7 @@ import torch
 from ..cache import CacheHandle, Request, StateRequest
 from ..kernels import ops
 from ..weights.binder import WeightSpec
-from .base import Mixer, Runtime, StepContext, emit_update, register_part
+from .base import Mixer, Runtime, StepContext, emit_update, register_part, update_operand
 
 
 @register_part("mixer", "mamba2")
@@ -265,5 +265,209 @@ class GatedDelta(Mixer):
         ctx.trace("scan", y)
         out = rt.empty(n, (self.v_width + 7) // 8 * 8)[:, : self.v_width]
         ops.head_norm_gate(y, gate, self.norm_w, self.eps, out, self.n_heads)
+        ctx.trace("attn", out)
+        return emit_update(out, self.w_o, ctx)
+
+
+@register_part("mixer", "mamba1")
+class Mamba1(Mixer):
+    """The selective scan with a decay per channel and state number (Mamba).
+
+    W_in x = [u: inner | z: inner]; u passes a causal convolution over the last
+    ``conv_taps`` tokens per channel, with a bias, and silu.  W_x u = [r: dt_rank |
+    B: N | C: N], dt = softplus(W_dt r + bias), one per channel.  Per channel c and
+    state n,
+
+        S[c, n] <- exp(-exp(a_log[c, n]) dt_c) S[c, n] + dt_c u_c B_n
+        y_c = sum_n S[c, n] C_n + d_c u_c
+
+    then y * silu(z) and the output projection.  What a sequence keeps between
+    steps is S and the last conv_taps - 1 inputs of the convolution, both float32
+    `StateRequest`s.  Step sizes, decays, the state and the sums are float32 in
+    both compute dtypes (W_dt leaves float32 sums); the projections, u, B and C are
+    in the compute dtype.  The reference has no recurrent mixer.
+
+    Parameters: ``hidden_size``, ``inner``, ``state_size``, ``dt_rank``,
+    ``conv_taps`` and the tensor names ``in``, ``conv``, ``conv_bias``, ``x``,
+    ``dt``, ``dt_bias``, ``a_log``, ``d``, ``o``.
+    """
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden = int(self.param("hidden_size"))
+        self.inner = int(self.param("inner"))
+        self.n_state = int(self.param("state_size"))
+        self.rank = int(self.param("dt_rank"))
+        self.taps = int(self.param("conv_taps"))
+        if self.taps < 1:
+            raise ValueError("the convolution needs at least one tap")
+        if self.n_state > ops.SELECTIVE_MAX_STATES:
+            raise ValueError(f"{self.n_state} states a channel are more than the scan's kernel takes ({ops.SELECTIVE_MAX_STATES})")
+        self.names = {k: str(self.param(k)) for k in ("in", "conv", "conv_bias", "x", "dt", "dt_bias", "a_log", "d", "o")}
+        self.rank_padded = (self.rank + 7) // 8 * 8
+        self.w_o: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        n, c = self.names, self.inner
+        return [WeightSpec(n["in"], (2 * c, self.hidden)),
+                WeightSpec(n["conv"], (c, self.taps), role="parameter", std=0.3),
+                WeightSpec(n["conv_bias"], (c,), role="parameter", std=0.1),
+                WeightSpec(n["x"], (self.rank + 2 * self.n_state, c)),
+                WeightSpec(n["dt"], (c, self.rank), std=0.1),
+                WeightSpec(n["dt_bias"], (c,), role="parameter", mean=-2.0, std=1.0),
+                WeightSpec(n["a_log"], (c, self.n_state), role="parameter", mean=0.5, std=0.8),
+                WeightSpec(n["d"], (c,), role="parameter", mean=1.0, std=0.3),
+                WeightSpec(n["o"], (self.hidden, c))]
+
+    def cache_requests(self) -> List[Request]:
+        requests: List[Request] = [StateRequest("scan", (self.inner, self.n_state), "float32")]
+        if self.taps > 1:
+            requests.append(StateRequest("conv", (self.taps - 1, self.inner), "float32"))
+        return requests
+
+    def last_product(self):
+        return self.names["o"], self.inner
+
+    def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        n = self.names
+        self.w_in = rt.matrix(tensors[n["in"]])
+        if not self.joined:
+            self.w_o = rt.matrix(tensors[n["o"]])
+        # the rows of r padded to a multiple of 8, so that B and C and the rows of W_dt's operand lie on
+        # the products' boundaries; the added rows and columns are zeros
+        w_x, w_dt = tensors[n["x"]].to(rt.dtype), tensors[n["dt"]].to(rt.dtype)
+        more = self.rank_padded - self.rank
+        if more:
+            w_x = torch.cat([w_x[: self.rank], w_x.new_zeros((more, self.inner)), w_x[self.rank:]], dim=0)
+            w_dt = torch.cat([w_dt, w_dt.new_zeros((self.inner, more))], dim=1)
+        self.w_x, self.w_dt = rt.matrix(w_x), rt.matrix(w_dt)
+        self.conv_w = rt.vector(tensors[n["conv"]].t().contiguous())      # tap by tap: [taps, channels]
+        self.conv_b = rt.vector(tensors[n["conv_bias"]])
+        self.dt_bias = rt.vector(tensors[n["dt_bias"]])
+        self.rates = rt.vector(-torch.exp(tensors[n["a_log"]].to(torch.float32)))
+        self.d = rt.vector(tensors[n["d"]])
+        self.no_state = torch.zeros((1, 0, self.inner), dtype=torch.float32, device=rt.device)
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        rt = ctx.rt
+        n = x.shape[0]
+        if not cache.writes:
+            raise ValueError("a recurrent mixer cannot read another run's state: every run advances its own")
+        padded = lambda width: (width + 7) // 8 * 8
+        proj = rt.empty(n, padded(2 * self.inner))[:, : 2 * self.inner]
+        ops.linear(x, self.w_in, proj)
+        u = rt.empty(n, padded(self.inner))[:, : self.inner]
+        conv_state = cache.state("conv") if self.taps > 1 else self.no_state
+        ops.causal_conv_silu(proj[:, : self.inner], self.conv_w, self.conv_b, conv_state, u, ctx.token_seq, ctx.cu_seqlens,
+                             ctx.slots, n_seqs=ctx.n_seqs, update_state=True, one_token_each=ctx.is_decode)
+        ctx.trace("conv", u)
+        low = rt.empty(n, padded(self.w_x.shape[0]))[:, : self.w_x.shape[0]]
+        ops.linear(u, self.w_x, low)
+        dt = rt.empty(n, padded(self.inner), dtype=torch.float32)[:, : self.inner]
+        ops.linear(low[:, : self.rank_padded], self.w_dt, dt)
+        out = update_operand(ctx, n, self.inner)
+        ops.selective_scan(u, low[:, self.rank_padded:], dt, self.dt_bias, self.rates, self.d, proj[:, self.inner:],
+                           cache.state("scan"), out, ctx.cu_seqlens, ctx.slots, ctx.n_seqs, one_token_each=ctx.is_decode)
+        ctx.trace("attn", out)
+        return emit_update(out, self.w_o, ctx)
+
+
+@register_part("mixer", "matrix_memory")
+class MatrixMemory(Mixer):
+    """The matrix memory with exponential input gates (mLSTM).
+
+    q = W_q x dim^-1/2 and k = W_k x (``n_heads`` heads of ``head_dim``), v = W_v x
+    (heads of ``value_dim``).  Per head a log input gate i = cap tanh((W_i x + b_i) /
+    cap), a log forget gate f = log sigmoid(cap tanh((W_f x + b_f) / cap)), cap =
+    ``gate_cap``, and
+
+        m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n likewise with k alone
+        o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+
+    S, n and m zero at the start.  Every head of o is divided by its root mean
+    square (``eps``), multiplied by a weight of all heads' channels and by
+    sigmoid(W_g x), and projected by W_o.  What a sequence keeps between steps is
+    S, n and m (m once per column of S and once for n: equal copies), float32
+    `StateRequest`s.  Gates, their logarithms and exponentials, the maximum, the
+    state, the sums and the norm are float32 in both compute dtypes (the gates'
+    projection leaves float32 sums); the other projections are in the compute
+    dtype.  The reference has no recurrent mixer.
+
+    Parameters: ``hidden_size``, ``n_heads``, ``head_dim``, ``value_dim``,
+    ``gate_cap``, ``eps`` and the tensor names ``q``, ``k``, ``v``, ``g``, ``i``,
+    ``i_bias``, ``f``, ``f_bias``, ``norm``, ``o``.
+    """
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden = int(self.param("hidden_size"))
+        self.n_heads = int(self.param("n_heads"))
+        self.dim = int(self.param("head_dim"))
+        self.vdim = int(self.param("value_dim"))
+        self.cap = float(self.param("gate_cap"))
+        self.eps = float(self.param("eps"))
+        if self.dim > ops.MLSTM_MAX_KEY_DIM:
+            raise ValueError(f"heads of {self.dim} key channels are more than the recurrence's kernel takes ({ops.MLSTM_MAX_KEY_DIM})")
+        self.names = {k: str(self.param(k)) for k in ("q", "k", "v", "g", "i", "i_bias", "f", "f_bias", "norm", "o")}
+        self.qk_width, self.v_width = self.n_heads * self.dim, self.n_heads * self.vdim
+        self.shares_input = False             # True once another part projects for this one
+        self.w_in: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        n, h = self.names, self.n_heads
+        return [WeightSpec(n["q"], (self.qk_width, self.hidden)), WeightSpec(n["k"], (self.qk_width, self.hidden)),
+                WeightSpec(n["v"], (self.v_width, self.hidden)), WeightSpec(n["g"], (self.v_width, self.hidden)),
+                WeightSpec(n["i"], (h, self.hidden)), WeightSpec(n["i_bias"], (h,), role="parameter", mean=-1.0, std=1.0),
+                WeightSpec(n["f"], (h, self.hidden)), WeightSpec(n["f_bias"], (h,), role="parameter", mean=3.0, std=1.0),
+                WeightSpec(n["norm"], (self.v_width,), role="vector", mean=1.0), WeightSpec(n["o"], (self.hidden, self.v_width))]
+
+    def cache_requests(self) -> List[Request]:
+        h = self.n_heads
+        return [StateRequest("memory", (h, self.dim, self.vdim), "float32"), StateRequest("normaliser", (h, self.dim), "float32"),
+                StateRequest("maximum", (h, self.vdim + 1), "float32")]
+
+    def input_matrix(self, tensors: Mapping[str, torch.Tensor]) -> List[torch.Tensor]:
+        """The matrices whose products with x, side by side, `forward_projected` reads."""
+        return [tensors[self.names[k]] for k in ("q", "k", "v", "g")]
+
+    @property
+    def input_width(self) -> int:
+        return 2 * (self.qk_width + self.v_width)
+
+    def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        n = self.names
+
+        def stacked(parts):
+            parts = [p.to(rt.dtype) for p in parts]
+            rows = sum(p.shape[0] for p in parts)
+            if rows % 8:
+                parts.append(parts[0].new_zeros((8 - rows % 8, self.hidden)))
+            return rt.matrix(torch.cat(parts, dim=0))
+        if not self.shares_input:
+            self.w_in = stacked(self.input_matrix(tensors))
+        self.w_gates = stacked([tensors[n["i"]], tensors[n["f"]]])
+        self.gate_bias = rt.vector(torch.cat([tensors[n[k]].reshape(-1).to(torch.float32) for k in ("i_bias", "f_bias")]))
+        self.norm_w = rt.vector(tensors[n["norm"]])
+        self.w_o = rt.matrix(tensors[n["o"]])
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        proj = ctx.rt.empty(x.shape[0], self.w_in.shape[0])
+        ops.linear(x, self.w_in, proj)
+        return self.forward_projected(proj[:, : self.input_width], x, ctx, cache)
+
+    def forward_projected(self, proj: torch.Tensor, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        rt, n, a, h = ctx.rt, x.shape[0], self.qk_width, self.n_heads
+        if not cache.writes:
+            raise ValueError("a recurrent mixer cannot read another run's state: every run advances its own")
+        gates = rt.empty(n, self.w_gates.shape[0], dtype=torch.float32)
+        ops.linear(x, self.w_gates, gates)
+        num = rt.empty(n, self.v_width, dtype=torch.float32)
+        den = rt.empty(n, h, dtype=torch.float32)
+        ops.mlstm_scan(proj[:, :a], proj[:, a: 2 * a], proj[:, 2 * a: 2 * a + self.v_width], gates[:, : 2 * h], self.gate_bias, self.cap,
+                       self.dim ** -0.5, tuple(cache.state(k) for k in ("memory", "normaliser", "maximum")), num, den, ctx.cu_seqlens,
+                       ctx.slots, ctx.n_seqs, h, one_token_each=ctx.is_decode)
+        ctx.trace("scan", num)
+        out = rt.empty(n, (self.v_width + 7) // 8 * 8)[:, : self.v_width]
+        ops.head_norm_gate(num, proj[:, 2 * a + self.v_width: 2 * (a + self.v_width)], self.norm_w, self.eps, out, h, den=den)
         ctx.trace("attn", out)
         return emit_update(out, self.w_o, ctx)
