@@ -86,7 +86,7 @@ class SwiGLU(FeedForward):
         # bfloat16: gate and up rows interleaved in blocks of 8 so that the product's
         # epilogue can apply silu(gate) * up to its float accumulators and write the
         # activation directly; float32: gate rows then up rows, and a kernel of its own
-        self.fused = (rt.dtype == torch.bfloat16 and self.inter % 8 == 0 and not self.bias_names
+        self.fused = (rt.dtype == torch.bfloat16 and self.inter % 8 == 0 and self.hidden % 8 == 0 and not self.bias_names
                       and self.activation in ops.GATED_EPILOGUES)
         if self.bias_names:
             self.biases = [rt.vector(tensors[name]) for name in self.bias_names]
