@@ -38,7 +38,11 @@ design (four copies of the hidden state, attention within stretches of
 positions, squared-relu experts; see `zotolix_shape`), and with --design megerax
 for the Megerax design (attention with convolved projections, capped scores and
 a gate on all channels, attention through a latent with sinks, the gated delta
-rule; see `megerax_shape`).  The default run is not changed by any of them.
+rule; see `megerax_shape`), and with --design mererax for the Mererax design
+(mixer and feed-forward side by side, the selective scan, attention with a
+penalty on the distance beside a matrix memory; see `mererax_shape`), which also
+measures the Ropovik design, the closest other one, beside it.  The default run
+is not changed by any of them.
 
 Peaks come from MEASURED_PEAKS.json beside this file if present, else from the
 fallback figures of an earlier measurement on the same pool.  Inputs are larger
@@ -524,6 +528,19 @@ def megerax_shape(width, heads, kv_heads, dim, ff, l_heads, l_rank, l_qrank, d_h
             "layers": four(0) + four(4)}
 
 
+def mererax_shape(width, heads, kv_heads, dim, ff, inner, state, rank, m_heads, m_dim, m_vdim, vocab=32000):
+    """Eight layers, a selective scan and a pair of mixers (attention whose values are the keys, beside a matrix memory)
+    in turn, each with a gated silu feed-forward beside it."""
+    mlp = {"kind": "dense", "ff": ff}
+    scan = {"type": "mamba1", "mixer": {"inner": inner, "state": state, "dt_rank": rank, "conv": 4}, "mlp": mlp}
+    pair = {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                               "q_temp": {"coef": 0.1, "every": 4096}},
+                      "right": {"heads": m_heads, "dim": m_dim, "vdim": m_vdim, "gate_cap": 15.0}}}
+    return {"architecture": "Mererax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+            "layers": [scan, pair] * 4}
+
+
 DESIGN_SIZES = {
     # the layer sizes of Llama-3.2-1B / SmolLM2 (width 2048) and of Llama-3.1-8B (width 4096); the
     # recurrence has twice the width in its inner size, heads of 64 and a state of 128, as Mamba-2 models do
@@ -549,7 +566,20 @@ MEGERAX_SIZES = {
     "w2048": (megerax_shape(2048, 32, 8, 64, 8192, 16, 512, 768, 16), dict(LLAMA_3P2_1B, num_hidden_layers=8, vocab_size=32000)),
     "w4096": (megerax_shape(4096, 32, 8, 128, 14336, 32, 512, 1536, 32), dict(LLAMA_3P1_8B, num_hidden_layers=8, vocab_size=32000)),
 }
+MERERAX_SIZES = {
+    # the same two widths, heads and feed-forward sizes as the Llama layers beside them; the scan has twice the width in
+    # its inner size and 16 states a channel, as Mamba models do, the memory eight heads whose values are as wide as the
+    # model together and twice as wide as its keys, as xLSTM models do; the third is the Ropovik design at equal size
+    "w2048": (mererax_shape(2048, 32, 8, 64, 8192, 4096, 16, 128, 8, 128, 256), dict(LLAMA_3P2_1B, num_hidden_layers=8, vocab_size=32000),
+              DESIGN_SIZES["w2048"][0]),
+    "w4096": (mererax_shape(4096, 32, 8, 128, 14336, 8192, 16, 256, 8, 256, 512), dict(LLAMA_3P1_8B, num_hidden_layers=8, vocab_size=32000),
+              DESIGN_SIZES["w4096"][0]),
+}
 DESIGNS = {
+    "mererax": (MERERAX_SIZES, "8 layers, a selective scan (16 states a channel) and a pair of mixers (attention with a penalty on the "
+                               "distance whose values are the keys, beside a matrix memory of eight heads) in turn, a gated silu "
+                               "feed-forward beside each mixer; beside 8 Llama layers of equal width, heads and feed-forward size and "
+                               "the Ropovik design (Mamba-2 and attention); vocabulary 32000"),
     "megerax": (MEGERAX_SIZES, "8 layers: attention with convolved projections, capped scores, a window of 1024 and a gate on all "
                                "channels (two with keys of their own, two reading theirs), attention through a latent with sinks, "
                                "the gated delta rule with heads of 128 x 128; a gated gelu feed-forward each; beside 8 Llama layers "
@@ -885,6 +915,137 @@ def run_design(args):
             del cache, kv_plain
         return rows
 
+    def mererax_kernel_table(cfg):
+        """Each kernel the Mererax design added or extended, alone, at this size: a prompt of T tokens
+        and a decode step of 64 sequences after 1,024 tokens; the bytes it has to move against the copy
+        peak and, for products and attention, its FLOPs against the matrix peak.  Beside each the like
+        kernel of the Llama or the Ropovik path at the same rows."""
+        from go_tinygrad_b200.cache import Cache, KVRequest
+        from go_tinygrad_b200.parts.base import StepContext
+        bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+        m, a, r = cfg["layers"][0]["mixer"], cfg["layers"][1]["mixer"]["left"], cfg["layers"][1]["mixer"]["right"]
+        H, ff, inner, N, rank, taps = cfg["width"], cfg["layers"][0]["mlp"]["ff"], m["inner"], m["state"], m["dt_rank"], m["conv"]
+        heads, n_kv, hd = a["heads"], a["kv_heads"], a["dim"]
+        mh, md, mv = r["heads"], r["dim"], r["vdim"]
+        rows = []
+
+        def add(name, rows_n, ms, nbytes, flops=0, like=None):
+            rows.append({"kernel": name, "rows": rows_n, "us": round(ms * 1e3, 2), "mb": round(nbytes / 1e6, 2),
+                         "of_copy_peak": round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3),
+                         **({"tflops": round(flops / ms / 1e9, 1), "of_matrix_peak": round(flops / ms / 1e9 / pk["bf16_tflops"], 3)} if flops else {}),
+                         **({"like": like} if like else {})})
+        rnd = lambda *shape, dtype=bf: torch.randn(*shape, device=dev, dtype=f32).to(dtype)
+        for n, n_seqs, ctx_len, tag in ((T, 1, 0, "prompt"), (64, 64, prompt_len, "decode")):
+            per = n // n_seqs
+            one = per == 1
+            rt = lib.parts.Runtime(dev, bf)
+            cache = Cache([[KVRequest(n_kv, hd, None)]], [None], max_tokens=64 * ((ctx_len + per + 63) // 64) * n_seqs, max_slots=n_seqs,
+                          dtype=bf, device=dev)
+            slot_list = [cache.open_sequence() for _ in range(n_seqs)]
+            cache.reserve_many([(s, ctx_len + per) for s in slot_list]); cache.flush_tables()
+            cache.groups[0].storage.normal_()
+            kv = cache.handles[0].kv
+            cu = torch.arange(0, n + 1, per, dtype=i32, device=dev)
+            seq = torch.arange(n, dtype=i32, device=dev) // per
+            slots = torch.tensor(slot_list, dtype=i32, device=dev)
+            start = torch.full((n_seqs,), ctx_len, dtype=i32, device=dev)
+            pos = (start[seq.long()] + (torch.arange(n, device=dev) % per)).to(i32)
+            ctx = StepContext(rt=rt, n_tokens=n, n_seqs=n_seqs, tokens=seq, positions=pos, token_seq=seq, cu_seqlens=cu, slots=slots,
+                              start_pos=start, max_q_len=per, max_kv_len=ctx_len + per, is_decode=one, total_kv_len=n_seqs * (ctx_len + per))
+            # embedding with sinusoids, beside without; two norms from one pass, beside one
+            table, res, upd, w = rnd(32000, H), rnd(n, H, dtype=f32), rnd(n, H), rnd(H, dtype=f32)
+            turns = torch.rand(H // 2, dtype=torch.float64, device=dev)
+            add(f"embed, sinusoids ({tag})", n, timed(lambda: ops.embed(seq, table, res, 8.0, pos, turns)), n * H * 6)
+            add(f"embed ({tag})", n, timed(lambda: ops.embed(seq, table, res, 8.0)), n * H * 6, like="embed, sinusoids")
+            out, out2 = torch.empty(n, H, dtype=bf, device=dev), torch.empty(n, H, dtype=bf, device=dev)
+            add(f"add_rmsnorm, two weights ({tag})", n, timed(lambda: ops.add_rmsnorm(res, upd, w, 1e-5, out, second=w, out_second=out2)), n * H * (4 + 4 + 2 + 4))
+            add(f"add_rmsnorm ({tag})", n, timed(lambda: ops.add_rmsnorm(res, upd, w, 1e-5, out)), n * H * (4 + 4 + 2 + 2), like="add_rmsnorm, two weights")
+            add(f"normed_pair ({tag})", n, timed(lambda: ops.normed_pair(upd, out, w, w, 1e-5, 0.5, residual=res)), n * H * (2 + 2 + 4 + 4))
+            add(f"rmsnorm_add ({tag})", n, timed(lambda: ops.rmsnorm_add(upd, w, 1e-5, res, out)), n * H * (2 + 4 + 4 + 2), like="normed_pair")
+            # norms over whole rows and cache store, beside rotation and cache store
+            C = (heads + n_kv) * hd
+            qk, nq, nk = rnd(n, C), rnd(heads * hd, dtype=f32), rnd(n_kv * hd, dtype=f32)
+            q = torch.empty(n, heads * hd, dtype=bf, device=dev)
+            add(f"qk_rows_finish ({tag})", n, timed(lambda: ops.qk_rows_finish(qk, nq, nk, 1e-5, heads, kv, q, seq, slots, pos, (0.1, 4096.0))),
+                n * (C + (heads + 2 * n_kv) * hd) * 2)
+            qkv, cs = rnd(n, C + n_kv * hd), rnd(n, hd // 2, 2, dtype=f32)
+            add(f"rope_kv_store ({tag})", n, timed(lambda: ops.rope_kv_store(qkv, cs, heads, n_kv, hd, kv, seq, slots, pos)),
+                n * (heads + 2 * n_kv) * hd * 4, like="qk_rows_finish")
+            # attention with a penalty on the distance, beside without, beside the decode attention of the Llama path
+            q.copy_(rnd(n, heads * hd))
+            mixed = torch.empty(n, heads * hd, dtype=bf, device=dev)
+            slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)], device=dev)
+            keys = n_seqs * (ctx_len + 1) if one else per * (per + 1) // 2
+            nbytes = n * heads * hd * 4 + n_seqs * n_kv * (ctx_len + per) * hd * 4
+            att = lambda **kw: timed(lambda: ops.attention_general(q, mixed, kv, ctx, heads, hd ** -0.5, **kw))
+            add(f"attention, sloped ({tag})", n, att(slopes=slopes), nbytes, 4 * heads * keys * hd)
+            add(f"attention, same kernel without slopes ({tag})", n, att(), nbytes, 4 * heads * keys * hd, like="attention, sloped")
+            if one:
+                splits, chunk, ring = ops.attention_decode_plan(n, heads, n_kv, hd, ctx_len + 1, 0, n * (ctx_len + 1))
+                scratch = torch.empty(max(1, ops.attention_decode_scratch_floats(n, heads, hd, splits)), dtype=f32, device=dev)
+                add(f"split-KV decode attention ({tag})", n,
+                    timed(lambda: ops.attention_decode_bf16(q, mixed, kv, slots, pos, heads, hd ** -0.5, 0, splits, scratch, chunk_pages=chunk, ring_pages=ring)),
+                    nbytes, 4 * heads * keys * hd, like="attention, sloped")
+            # the matrix memory: recurrence, division, norm and gate; beside the state-space recurrence of the Ropovik
+            # path at as many state numbers
+            wide = rnd(n, 2 * mh * (md + mv))
+            gates, gb = rnd(n, 2 * mh, dtype=f32), torch.cat([torch.zeros(mh), torch.full((mh,), 4.0)]).to(dev)
+            st = (torch.zeros(n_seqs, mh, md, mv, device=dev), torch.zeros(n_seqs, mh, md, device=dev), torch.zeros(n_seqs, mh, mv + 1, device=dev))
+            num, den = torch.empty(n, mh * mv, dtype=f32, device=dev), torch.empty(n, mh, dtype=f32, device=dev)
+            qk_w = mh * md
+            add(f"mlstm_scan ({tag})", n,
+                timed(lambda: ops.mlstm_scan(wide[:, :qk_w], wide[:, qk_w:2 * qk_w], wide[:, 2 * qk_w:2 * qk_w + mh * mv], gates, gb, 15.0, md ** -0.5,
+                                             st, num, den, cu, slots, n_seqs, mh, one_token_each=one)),
+                n * (2 * qk_w * 2 + mh * mv * (2 + 4) + 3 * mh * 4) + n_seqs * mh * md * mv * 8)
+            nw, om = rnd(mh * mv, dtype=f32), torch.empty(n, mh * mv, dtype=bf, device=dev)
+            add(f"head_norm_gate, divided ({tag})", n, timed(lambda: ops.head_norm_gate(num, wide[:, 2 * qk_w + mh * mv:], nw, 1e-5, om, mh, den=den)),
+                n * mh * mv * (4 + 2 + 2))
+            sh, sp, sn, sg = mh * md * mv // (64 * 128), 64, 128, 8
+            xs, bc = rnd(n, sh * sp), rnd(n, sg * sn, 2, dtype=f32)
+            dt_raw, dtb, alog, skip = rnd(n, sh), rnd(sh, dtype=f32), rnd(sh, dtype=f32), rnd(sh, dtype=f32)
+            S2, y2 = torch.zeros(n_seqs, sh, sn, sp, device=dev), torch.empty(n, sh * sp, dtype=f32, device=dev)
+            add(f"ssm_scan, as many state numbers ({tag})", n,
+                timed(lambda: ops.ssm_scan(xs, bc, dt_raw, dtb, alog, skip, S2, y2, cu, slots, n_seqs, sh, sg, sn, sp, one_token_each=one)),
+                n * (sh * sp * 6 + sg * sn * 8) + n_seqs * sh * sn * sp * 8, like="mlstm_scan")
+            zz, og = rnd(n, mh * mv), torch.empty(n, mh * mv, dtype=bf, device=dev)
+            add(f"gated_rmsnorm ({tag})", n, timed(lambda: ops.gated_rmsnorm(num, zz, nw, 1e-5, og, mh)), n * mh * mv * (4 + 2 + 2), like="head_norm_gate, divided")
+            # the selective scan with its gate; beside the state-space recurrence and its gated norm at equal inner size
+            proj, low = rnd(n, 2 * inner), rnd(n, 2 * N)
+            dt, dbias, skip1 = rnd(n, inner, dtype=f32), rnd(inner, dtype=f32) - 3, rnd(inner, dtype=f32)
+            rates, S1 = -torch.rand(inner, N, device=dev) * 4, torch.zeros(n_seqs, inner, N, device=dev)
+            cw, cb, cst = rnd(taps, inner, dtype=f32), rnd(inner, dtype=f32), torch.zeros(n_seqs, taps - 1, inner, device=dev)
+            u, oi = torch.empty(n, inner, dtype=bf, device=dev), torch.empty(n, inner, dtype=bf, device=dev)
+            add(f"causal_conv_silu ({tag})", n,
+                timed(lambda: ops.causal_conv_silu(proj[:, :inner], cw, cb, cst, u, seq, cu, slots, n_seqs=n_seqs, update_state=True, one_token_each=one)),
+                n * inner * 4 + (n_seqs * (taps - 1) * inner * 8 if one else 0))
+            add(f"selective_scan ({tag})", n,
+                timed(lambda: ops.selective_scan(u, low, dt, dbias, rates, skip1, proj[:, inner:], S1, oi, cu, slots, n_seqs, one_token_each=one)),
+                n * (inner * (2 + 4 + 2 + 2) + 2 * N * 2) + n_seqs * inner * N * 8)
+            sh = inner // 64
+            xs, bc, dt_raw = rnd(n, inner), rnd(n, sg * sn, 2, dtype=f32), rnd(n, sh)
+            dtb, alog, skip = rnd(sh, dtype=f32), rnd(sh, dtype=f32), rnd(sh, dtype=f32)
+            S2, y2 = torch.zeros(n_seqs, sh, sn, sp, device=dev), torch.empty(n, inner, dtype=f32, device=dev)
+            add(f"ssm_scan, equal inner size ({tag})", n,
+                timed(lambda: ops.ssm_scan(xs, bc, dt_raw, dtb, alog, skip, S2, y2, cu, slots, n_seqs, sh, sg, sn, sp, one_token_each=one)),
+                n * (inner * 6 + sg * sn * 8) + n_seqs * sh * sn * sp * 8, like="selective_scan")
+            # products: the joint one beside the feed-forward's own, the two narrow ones of the scan, the gates'
+            x = rnd(n, H)
+            product = lambda xx, ww, o: timed(lambda: ops.linear(xx, ww, o))
+            for label, K, M, dtype, like in (("joint product of mixer and feed-forward", inner + ff, H, bf, None), ("down product alone", ff, H, bf, "joint product"),
+                                             ("product to dt, B and C", inner, rank + 2 * N, bf, None), ("product of dt", rank, inner, f32, None),
+                                             ("product of the memory's gates", H, 2 * mh, f32, None),
+                                             ("product of both mixers' inputs", H, C + 2 * mh * (md + mv), bf, None)):
+                xx, ww, o = rnd(n, K), rnd(M, K), torch.empty(n, M, dtype=dtype, device=dev)
+                if label.startswith(("joint", "down")) and not one:
+                    ms = timed(lambda: ops.linear_add_residual(xx, ww, res))
+                    nbytes = (n * K + M * K) * 2 + n * M * 8
+                else:
+                    ms = product(xx, ww, o)
+                    nbytes = (n * K + M * K) * 2 + n * M * o.element_size()
+                add(f"{label} ({tag})", n, ms, nbytes, 2 * n * M * K, like=like)
+            del cache
+        return rows
+
     def zotolix_kernel_table(cfg):
         """Each kernel the Zotolix design added or extended, alone, at this size: a prompt of T
         tokens and a decode step of 64 sequences at the last place of a stretch; the bytes it has to move
@@ -1058,10 +1219,12 @@ def run_design(args):
     sampler.mark()
     sizes = {}
     design_sizes, what = DESIGNS[args.design]
-    table = {"senupel": senupel_kernel_table, "zotolix": zotolix_kernel_table, "megerax": megerax_kernel_table}.get(args.design, kernel_table)
+    table = {"senupel": senupel_kernel_table, "zotolix": zotolix_kernel_table, "megerax": megerax_kernel_table,
+             "mererax": mererax_kernel_table}.get(args.design, kernel_table)
     for name in (args.sizes.split(",") if args.sizes else list(design_sizes)):
-        design_cfg, llama_cfg = design_sizes[name]
+        design_cfg, llama_cfg, *closest = design_sizes[name]
         sizes[name] = {args.design: model_numbers(design_cfg), "llama": model_numbers(llama_cfg),
+                       **{cfg["architecture"].lower(): model_numbers(cfg) for cfg in closest},
                        "kernels": table(design_cfg)}
     clocks = sampler.stop()
     print(json.dumps({"design": args.design, "dtype": "bf16", "data": "synthetic (random weights and token ids)",
