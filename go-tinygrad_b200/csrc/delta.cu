@@ -457,6 +457,80 @@ head_norm_gate_kernel(const float* __restrict__ y, int ld_y, const G* __restrict
     for (int c = lane; c < dv; c += 32)
         dst[c] = from_f32<T>(src[c] * inv * w[c] * (1.0f / (1.0f + expf(-to_f32<G>(gt[c])))));
 }
+
+// four neighbouring channels in one access
+__device__ __forceinline__ float4 load_four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_four(const bf16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(bf16* p, float4 v) {
+    uint2 o;
+    *reinterpret_cast<__nv_bfloat162*>(&o.x) = __floats2bfloat162_rn(v.x, v.y);
+    *reinterpret_cast<__nv_bfloat162*>(&o.y) = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = o;
+}
+
+// The same where rows, heads and addresses allow it: a lane takes four neighbouring channels at a time, KV such
+// pieces (dv <= 128 KV), all of whose loads are in flight together; the head is read once.
+template <typename T, typename G, int KV>
+__global__ void __launch_bounds__(256)
+head_norm_gate_vec_kernel(const float* __restrict__ y, int ld_y, const G* __restrict__ gate, int ld_gate,
+                          const float* __restrict__ weight, int w_step, float eps, const float* __restrict__ den,
+                          T* __restrict__ out, int ld_out, long long n_items, int n_heads, int dv) {
+    chain_release();
+    chain_wait();
+    const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (item >= n_items) return;
+    const int lane = threadIdx.x & 31;
+    const size_t n = (size_t)(item / n_heads);
+    const int h = (int)(item % n_heads);
+    const float* src = y + n * ld_y + (size_t)h * dv;
+    const G* gt = gate + n * ld_gate + (size_t)h * dv;
+    const float* w = weight + (size_t)h * w_step;
+    float4 v[KV], g[KV];
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        const int c = (lane + 32 * k) * 4;
+        v[k] = c < dv ? load_four(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        g[k] = c < dv ? load_four(gt + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float part = den ? 1.0f / den[item] : 1.0f;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        v[k].x *= part; v[k].y *= part; v[k].z *= part; v[k].w *= part;
+        ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
+    T* dst = out + n * ld_out + (size_t)h * dv;
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        const int c = (lane + 32 * k) * 4;
+        if (c >= dv) continue;
+        const float4 ww = load_four(w + c);
+        store_four(dst + c, make_float4(v[k].x * inv * ww.x / (1.0f + expf(-g[k].x)), v[k].y * inv * ww.y / (1.0f + expf(-g[k].y)),
+                                        v[k].z * inv * ww.z / (1.0f + expf(-g[k].z)), v[k].w * inv * ww.w / (1.0f + expf(-g[k].w))));
+    }
+}
+
+template <typename T, typename G>
+static int launch_head_norm_gate(const float* y, int ld_y, const void* gate, int ld_gate, const float* weight, int w_step, float eps,
+                                 const float* den, void* out, int ld_out, long long items, int n_heads, int dv, cudaStream_t stream) {
+    const dim3 grid((unsigned)((items + 7) / 8));
+    const bool fours = dv % 4 == 0 && ld_y % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && ((uintptr_t)y % 16) == 0 &&
+                       ((uintptr_t)weight % 16) == 0 && ((uintptr_t)gate % (4 * sizeof(G))) == 0 && ((uintptr_t)out % (4 * sizeof(T))) == 0;
+#define GTG_HEAD_NORM(KERNEL)                                                                                        \
+    return launch_chained(KERNEL, grid, dim3(256), 0, stream, y, ld_y, (const G*)gate, ld_gate, weight, w_step, eps, den, (T*)out, \
+                          ld_out, items, n_heads, dv)
+    if (fours && dv <= 128) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 1>));
+    if (fours && dv <= 256) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 2>));
+    if (fours && dv <= 512) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 4>));
+    GTG_HEAD_NORM((head_norm_gate_kernel<T, G>));
+#undef GTG_HEAD_NORM
+}
 }  // namespace
 
 GTG_API int gtg_delta_prepare(float* qk, int ld_qk, float* decay, int ld_decay, const float* dt_bias, const float* a_log,
@@ -551,14 +625,9 @@ GTG_API int gtg_head_norm_gate(int dtype, int gate_f32, const float* y, int ld_y
     const long long items = (long long)N * n_heads;
     const long long blocks = (items + 7) / 8;
     if (blocks > 0x7fffffffLL) return kErrUnsupported;
-    if (dtype == 0 && gate_f32)
-        return launch_chained(head_norm_gate_kernel<float, float>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const float*)gate,
-                              ld_gate, weight, w_step, eps, den, (float*)out, ld_out, items, n_heads, dv);
-    if (dtype == 1 && gate_f32)
-        return launch_chained(head_norm_gate_kernel<bf16, float>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const float*)gate,
-                              ld_gate, weight, w_step, eps, den, (bf16*)out, ld_out, items, n_heads, dv);
-    if (dtype == 1)
-        return launch_chained(head_norm_gate_kernel<bf16, bf16>, dim3((unsigned)blocks), dim3(256), 0, stream, y, ld_y, (const bf16*)gate,
-                              ld_gate, weight, w_step, eps, den, (bf16*)out, ld_out, items, n_heads, dv);
+#define GTG_ARGS y, ld_y, gate, ld_gate, weight, w_step, eps, den, out, ld_out, items, n_heads, dv, stream
+    if (dtype == 0 && gate_f32) return launch_head_norm_gate<float, float>(GTG_ARGS);
+    if (dtype == 1) return gate_f32 ? launch_head_norm_gate<bf16, float>(GTG_ARGS) : launch_head_norm_gate<bf16, bf16>(GTG_ARGS);
+#undef GTG_ARGS
     return kErrBadArgument;
 }

@@ -49,61 +49,71 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
 }
 
 // ------------------------------------------------ prompts: the recurrence token by token
-// One block per (head, slice of columns, sequence).  A warp serves CP neighbouring columns
-// over all rows: lane l owns KR rows in runs of V = min(KR, 4), rows V (l + 32 j) .. + V,
-// so that k and q of a token arrive by 8- or 16-byte reads from shared memory (rows beyond
-// d are zeros there).  Tiles of kTT tokens are staged as floats, the loads of the next tile
-// in flight meanwhile; a warp of its own works out the gates of the tile ahead.  The sums of
-// four tokens and CP columns meet in one butterfly in which every exchange halves what a
-// lane still carries.  Tokens are walked strictly in order: the result does not depend on
-// the cut of the sequence into steps, on the batch or on the slices.
+// One block per (head, slice of columns, sequence).  RG lanes share kCP neighbouring columns,
+// each owning kKR rows of them in registers: rows 4 (r + RG j) .. + 4 for lane r of the RG, so
+// that k and q of a token arrive by 16-byte reads from shared memory (rows beyond d are zeros
+// there).  A warp serves 32 / RG such groups.  What a token costs a lane is kKR kCP products and
+// two fused multiply-adds each, on pairs of rows; the sums of four tokens and kCP columns meet in
+// one butterfly in which every exchange halves what a lane still carries.
+//
+// Tiles of kTT tokens are double-buffered in shared memory as floats.  While the columns' warps
+// compute a tile, four warps of helpers store the next one (its loads were issued a tile earlier)
+// and write the results of the one before to memory, and one warp works out the gates of the next.
+// A token beyond the last is staged as zeros with a step that changes nothing.  Tokens are walked
+// strictly in order: the result does not depend on the cut of the sequence into steps, on the
+// batch or on the slices.
 constexpr int kTT = 16;
-constexpr int kMaxWarps = 8;
+constexpr int kKR = 16;                    // rows a lane owns
+constexpr int kCP = 2;                     // columns a lane owns
+constexpr int kMaxWarps = 8;               // warps of columns a block may have
+constexpr int kHelpers = 128;              // threads that move tiles
+constexpr int kMaxCols = 64;               // columns a block may serve
 
-template <typename T, int KR, int CP>
-__global__ void __launch_bounds__((kMaxWarps + 1) * 32)
+template <typename T, int RG>
+__global__ void __launch_bounds__(kMaxWarps * 32 + 32 + kHelpers)
 mlstm_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, int ld,
                   const float* __restrict__ gates, int ld_gates, const float* __restrict__ gate_bias, float cap, float q_scale,
                   float* __restrict__ S_all, float* __restrict__ n_all, float* __restrict__ m_all,
                   float* __restrict__ num, int ld_num, float* __restrict__ den,
-                  const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int heads, int d, int dv, int slices, int vec) {
+                  const int* __restrict__ cu_seqlens, const int* __restrict__ slots, int heads, int d, int dv, int warps, int slices, int vec) {
     chain_release();
     chain_wait();
-    constexpr int D = 32 * KR, V = KR < 4 ? KR : 4, P = KR / 2;
+    constexpr int D = RG * kKR, WC = 32 / RG * kCP;
     extern __shared__ __align__(16) float smem[];
-    const int warps = (blockDim.x >> 5) - 1, cols = warps * CP, threads = warps * 32;
-    float* sk = smem;                              // [kTT][D]
-    float* sq = sk + kTT * D;                      // [kTT][D]
-    float* sv = sq + kTT * D;                      // [kTT][cols], times the token's input factor
-    float* sy = sv + kTT * cols;                   // [kTT][cols]
-    float4* sg = reinterpret_cast<float4*>(sy + kTT * cols);     // two tiles of [kTT] (keep, add, exp(-m), m)
+    const int cols = warps * WC;
+    float* sk = smem;                              // [2][kTT][D]
+    float* sq = sk + 2 * kTT * D;                  // [2][kTT][D]
+    float* sv = sq + 2 * kTT * D;                  // [2][kTT][cols]
+    float* sy = sv + 2 * kTT * cols;               // [2][kTT][cols]
+    float4* sg = reinterpret_cast<float4*>(sy + 2 * kTT * cols);     // [2][kTT] (keep, add, exp(-m), m)
     const int h = blockIdx.x / slices, slice = blockIdx.x % slices, b = blockIdx.y;
     const int first = cu_seqlens[b], last = cu_seqlens[b + 1];
     if (first >= last) return;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int j0 = slice * cols;                   // the block's first column
+    const int tiles = (last - first + kTT - 1) / kTT;
     const size_t head = (size_t)slots[b] * heads + h;
-    float* S = S_all + head * d * dv;
-    float* nn = n_all + head * d;
     float* mm = m_all + head * (dv + 1);
 
     if (warp == warps) {
         // ---------------------------------------------------------------- the gates' warp
         float m = mm[j0];
         const float bi = gate_bias[h], bf = gate_bias[heads + h];
-        auto read = [&](int t0, float& ri, float& rf) {
+        float ri = 0.f, rf = 0.f;
+        auto read = [&](int t0) {
             const bool ok = lane < kTT && t0 + lane < last;
             const float* g = gates + (size_t)(ok ? t0 + lane : first) * ld_gates;
             ri = ok ? g[h] : 0.f;
             rf = ok ? g[heads + h] : 0.f;
         };
-        auto work = [&](int t0, int stage, float ri, float rf) {
+        auto work = [&](int t0, int stage) {
             const float i = capped(ri + bi, cap), f = log_sigmoid_f(capped(rf + bf, cap));
             const int nt = min(kTT, last - t0);
             float m_before = 0.f, m_after = 0.f;
-            for (int t = 0; t < nt; ++t) {
+#pragma unroll
+            for (int t = 0; t < kTT; ++t) {
                 const float ft = __shfl_sync(0xffffffffu, f, t), it = __shfl_sync(0xffffffffu, i, t);
-                const float next = fmaxf(ft + m, it);
+                const float next = t < nt ? fmaxf(ft + m, it) : m;
                 if (lane == t) { m_before = m; m_after = next; }
                 m = next;
             }
@@ -111,190 +121,212 @@ mlstm_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __r
                 sg[stage * kTT + lane] = lane < nt ? make_float4(expf(f + m_before - m_after), expf(i - m_after), expf(-m_after), m_after)
                                                    : make_float4(1.f, 0.f, 1.f, 0.f);
         };
-        float ri, rf;
-        read(first, ri, rf);
-        work(first, 0, ri, rf);
-        int stage = 0;
-        read(first + kTT, ri, rf);
-        for (int t0 = first; t0 < last; t0 += kTT, stage ^= 1) {
-            __syncthreads();                       // (1) the tile before has been computed; this tile's gates stand
-            __syncthreads();                       // (2) this tile is staged
-            if (t0 + kTT < last) {
-                work(t0 + kTT, stage ^ 1, ri, rf);
-                read(t0 + 2 * kTT, ri, rf);
+        read(first);
+        work(first, 0);
+        read(first + kTT);
+        __syncthreads();
+        for (int t = 0; t < tiles; ++t) {
+            if (t + 1 < tiles) {
+                work(first + (t + 1) * kTT, (t + 1) & 1);
+                read(first + (t + 2) * kTT);
             }
+            __syncthreads();
         }
         for (int c = lane; c < cols; c += 32)
             if (j0 + c <= dv) mm[j0 + c] = m;
         return;
     }
 
-    // ------------------------------------------------------------------ the columns' warps
-    const int wc = warp * CP;                      // the warp's first column within the slice
-    f32x2 s[CP][P];
+    if (warp > warps) {
+        // --------------------------------------------------------------- the helpers' warps
+        const int tid = threadIdx.x - (warps + 1) * 32;
+        constexpr int kPieces = 2 * kTT * (D / 8) / kHelpers;      // 8 elements each: k rows of the tile, then q rows
+        constexpr int kValues = kTT * kMaxCols / kHelpers;
+        uint4 raw[kPieces];
+        T rv[kValues];
+        // (token, column) of this thread's first value, and what the next one adds
+        const int v_tt = tid / cols, v_c = tid % cols, v_dt = kHelpers / cols, v_dc = kHelpers % cols;
+        auto fetch = [&](int t0) {
+            int tt = v_tt, c = v_c;
 #pragma unroll
-    for (int c = 0; c < CP; ++c) {
+            for (int e = 0; e < kValues; ++e) {
+                if (tt < kTT) {
+                    const int col = j0 + c;
+                    rv[e] = (t0 + tt < last && col < dv) ? v[(size_t)(t0 + tt) * ld + (size_t)h * dv + col] : from_f32<T>(col == dv ? 1.f : 0.f);
+                }
+                tt += v_dt;
+                c += v_dc;
+                if (c >= cols) { c -= cols; ++tt; }
+            }
+            if constexpr (sizeof(T) == 2) {
+                if (!vec) return;
+#pragma unroll
+                for (int e = 0; e < kPieces; ++e) {
+                    const int idx = tid + e * kHelpers, which = idx / (kTT * (D / 8)), rest = idx % (kTT * (D / 8));
+                    const int tt = rest / (D / 8), at = (rest % (D / 8)) * 8;
+                    raw[e] = (t0 + tt < last && at < d) ? *reinterpret_cast<const uint4*>((which ? q : k) + (size_t)(t0 + tt) * ld + (size_t)h * d + at)
+                                                        : make_uint4(0u, 0u, 0u, 0u);
+                }
+            }
+        };
+        auto store = [&](int t0, int stage) {
+            float* dk = sk + stage * kTT * D;
+            float* dq = sq + stage * kTT * D;
+#pragma unroll
+            for (int e = 0; e < kValues; ++e) {
+                const int idx = tid + e * kHelpers;
+                if (idx < kTT * cols) sv[stage * kTT * cols + idx] = to_f32<T>(rv[e]);
+            }
+            if constexpr (sizeof(T) == 2) {
+                if (vec) {
+#pragma unroll
+                    for (int e = 0; e < kPieces; ++e) {
+                        const int idx = tid + e * kHelpers, which = idx / (kTT * (D / 8)), rest = idx % (kTT * (D / 8));
+                        float* dst = (which ? dq : dk) + rest * 8;
+                        const float factor = which ? q_scale : 1.f;
+                        const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[e]);
+                        const float2 a0 = __bfloat1622float2(h2[0]), a1 = __bfloat1622float2(h2[1]);
+                        const float2 a2 = __bfloat1622float2(h2[2]), a3 = __bfloat1622float2(h2[3]);
+                        reinterpret_cast<float4*>(dst)[0] = make_float4(a0.x * factor, a0.y * factor, a1.x * factor, a1.y * factor);
+                        reinterpret_cast<float4*>(dst)[1] = make_float4(a2.x * factor, a2.y * factor, a3.x * factor, a3.y * factor);
+                    }
+                    return;
+                }
+            }
+            for (int idx = tid; idx < kTT * D; idx += kHelpers) {
+                const int tt = idx / D, at = idx % D;
+                const bool ok = t0 + tt < last && at < d;
+                const size_t where = ok ? (size_t)(t0 + tt) * ld + (size_t)h * d + at : 0;
+                dk[idx] = ok ? to_f32<T>(k[where]) : 0.f;
+                dq[idx] = ok ? to_f32<T>(q[where]) * q_scale : 0.f;
+            }
+        };
+        auto show = [&](int t) {                   // tile t's results to memory
+            const int t0 = first + t * kTT, nt = min(kTT, last - t0);
+            int tt = v_tt, c = v_c;
+            for (int idx = tid; idx < nt * cols; idx += kHelpers) {
+                const size_t row = (size_t)(t0 + tt);
+                const float x = sy[(t & 1) * kTT * cols + idx];
+                if (j0 + c < dv) num[row * ld_num + (size_t)h * dv + j0 + c] = x;
+                else if (j0 + c == dv) den[row * heads + h] = x;
+                tt += v_dt;
+                c += v_dc;
+                if (c >= cols) { c -= cols; ++tt; }
+            }
+        };
+        fetch(first);
+        store(first, 0);
+        if (tiles > 1) fetch(first + kTT);
+        __syncthreads();
+        for (int t = 0; t < tiles; ++t) {
+            if (t + 1 < tiles) {
+                store(first + (t + 1) * kTT, (t + 1) & 1);
+                if (t + 2 < tiles) fetch(first + (t + 2) * kTT);
+            }
+            if (t > 0) show(t - 1);
+            __syncthreads();
+        }
+        show(tiles - 1);
+        return;
+    }
+
+    // ------------------------------------------------------------------ the columns' warps
+    const int r = lane % RG, wc = warp * WC + lane / RG * kCP;       // the lane's rows, its first column within the slice
+    float* S = S_all + head * d * dv;
+    float* nn = n_all + head * d;
+    f32x2 s[kCP][kKR / 2];
+#pragma unroll
+    for (int c = 0; c < kCP; ++c) {
         const int col = j0 + wc + c;
 #pragma unroll
-        for (int p = 0; p < P; ++p) {
+        for (int p = 0; p < kKR / 2; ++p) {
             float e[2];
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
-                const int i = 2 * p + x, row = (i / V) * 32 * V + lane * V + i % V;
+                const int i = 2 * p + x, row = i / 4 * 4 * RG + r * 4 + i % 4;
                 e[x] = (row < d && col < dv) ? S[(size_t)row * dv + col] : (row < d && col == dv) ? nn[row] : 0.f;
             }
             s[c][p] = pair_of(e[0], e[1]);
         }
     }
-    // staging by pieces of 8 elements (16 bytes of bfloat16): piece e of this thread is number tid + e threads
-    // of the tile's k rows, then of its q rows
-    constexpr int kMaxPieces = 2 * kTT * D / 8 / 128;        // (with four warps; half of them with eight)
-    uint4 raw[kMaxPieces];
-    T rv[CP / 2];                                  // the tile's values: kTT cols of them over all threads
-    auto fetch = [&](int t0) {
-#pragma unroll
-        for (int e = 0; e < CP / 2; ++e) {
-            const int idx = tid + e * threads, tt = idx / cols, col = j0 + idx % cols;
-            rv[e] = (t0 + tt < last && col < dv) ? v[(size_t)(t0 + tt) * ld + (size_t)h * dv + col]
-                                                 : from_f32<T>(t0 + tt < last && col == dv ? 1.f : 0.f);
-        }
-        if constexpr (sizeof(T) == 2) {
-            if (!vec) return;
-#pragma unroll
-            for (int e = 0; e < kMaxPieces; ++e) {
-                const int idx = tid + e * threads;
-                raw[e] = make_uint4(0u, 0u, 0u, 0u);
-                if (idx >= 2 * kTT * (D / 8)) continue;
-                const int which = idx / (kTT * (D / 8)), rest = idx % (kTT * (D / 8));
-                const int tt = rest / (D / 8), at = (rest % (D / 8)) * 8;
-                if (t0 + tt < last && at < d)
-                    raw[e] = *reinterpret_cast<const uint4*>((which ? q : k) + (size_t)(t0 + tt) * ld + (size_t)h * d + at);
-            }
-        }
-    };
-    fetch(first);
-    int stage = 0, shown = first, shown_n = 0;     // the tile whose results lie in sy
-    auto show = [&]() {
-        for (int idx = tid; idx < shown_n * cols; idx += threads) {
-            const int tt = idx / cols, c = idx % cols;
-            const size_t row = (size_t)(shown + tt);
-            if (j0 + c < dv) num[row * ld_num + (size_t)h * dv + j0 + c] = sy[idx];
-            else if (j0 + c == dv) den[row * heads + h] = sy[idx];
-        }
-    };
-    for (int t0 = first; t0 < last; t0 += kTT, stage ^= 1) {
-        const int nt = min(kTT, last - t0);
-        __syncthreads();                           // (1)
-        show();
-        if constexpr (sizeof(T) == 2) {
-            if (vec) {
-#pragma unroll
-                for (int e = 0; e < kMaxPieces; ++e) {
-                    const int idx = tid + e * threads;
-                    if (idx >= 2 * kTT * (D / 8)) continue;
-                    const int which = idx / (kTT * (D / 8)), rest = idx % (kTT * (D / 8));
-                    float* dst = (which ? sq : sk) + rest * 8;
-                    const float factor = which ? q_scale : 1.f;
-                    const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&raw[e]);
-                    const float2 a = __bfloat1622float2(h2[0]), bb = __bfloat1622float2(h2[1]);
-                    const float2 c = __bfloat1622float2(h2[2]), dd = __bfloat1622float2(h2[3]);
-                    reinterpret_cast<float4*>(dst)[0] = make_float4(a.x * factor, a.y * factor, bb.x * factor, bb.y * factor);
-                    reinterpret_cast<float4*>(dst)[1] = make_float4(c.x * factor, c.y * factor, dd.x * factor, dd.y * factor);
-                }
-            }
-        }
-        if (sizeof(T) == 4 || !vec) {
-            for (int idx = tid; idx < kTT * D; idx += threads) {
-                const int tt = idx / D, at = idx % D;
-                const bool ok = tt < nt && at < d;
-                const size_t where = ok ? (size_t)(t0 + tt) * ld + (size_t)h * d + at : 0;
-                sk[idx] = ok ? to_f32<T>(k[where]) : 0.f;
-                sq[idx] = ok ? to_f32<T>(q[where]) * q_scale : 0.f;
-            }
-        }
-#pragma unroll
-        for (int e = 0; e < CP / 2; ++e) {
-            const int idx = tid + e * threads;
-            sv[idx] = to_f32<T>(rv[e]) * sg[stage * kTT + idx / cols].y;
-        }
-        __syncthreads();                           // (2)
-        if (t0 + kTT < last) fetch(t0 + kTT);
-        for (int tq = 0; tq < nt; tq += 4) {
-            float part[4 * CP];
+    __syncthreads();
+    for (int t = 0; t < tiles; ++t) {
+        const int stage = t & 1;
+        const float* tk = sk + stage * kTT * D + r * 4;
+        const float* tq = sq + stage * kTT * D + r * 4;
+        const float* tv = sv + stage * kTT * cols + wc;
+        const float4* tg = sg + stage * kTT;
+#pragma unroll 1
+        for (int t4 = 0; t4 < kTT; t4 += 4) {
+            constexpr int kSums = 4 * kCP;
+            float part[kSums];
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-                const float keep = sg[stage * kTT + tq + u].x;
-                const f32x2 keep2 = pair_of(keep, keep);
-                f32x2 val[CP], acc[CP];
+                const float4 g = tg[t4 + u];
+                const f32x2 keep = pair_of(g.x, g.x);
+                f32x2 val[kCP], acc[kCP];
+                float vv[kCP];
+                *reinterpret_cast<float2*>(vv) = *reinterpret_cast<const float2*>(tv + (t4 + u) * cols);
 #pragma unroll
-                for (int c = 0; c < CP; ++c) {
-                    const float x = sv[(tq + u) * cols + wc + c];
+                for (int c = 0; c < kCP; ++c) {
+                    const float x = vv[c] * g.y;
                     val[c] = pair_of(x, x);
                     acc[c] = pair_of(0.f, 0.f);
                 }
 #pragma unroll
-                for (int run = 0; run < KR / V; ++run) {
-                    f32x2 kk[V / 2], qq[V / 2];
-                    const int at = (tq + u) * D + run * 32 * V + lane * V;
-                    if constexpr (V == 4) {
-                        const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(sk + at), e = *reinterpret_cast<const ulonglong2*>(sq + at);
-                        kk[0] = a.x; kk[1] = a.y; qq[0] = e.x; qq[1] = e.y;
-                    } else {
-                        kk[0] = *reinterpret_cast<const f32x2*>(sk + at);
-                        qq[0] = *reinterpret_cast<const f32x2*>(sq + at);
-                    }
+                for (int j = 0; j < kKR / 4; ++j) {
+                    const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(tk + (t4 + u) * D + j * 4 * RG);
+                    const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(tq + (t4 + u) * D + j * 4 * RG);
 #pragma unroll
-                    for (int p = 0; p < V / 2; ++p) {
-#pragma unroll
-                        for (int c = 0; c < CP; ++c) {
-                            f32x2& x = s[c][run * (V / 2) + p];
-                            x = fma2(keep2, x, mul2(kk[p], val[c]));
-                            acc[c] = fma2(x, qq[p], acc[c]);
-                        }
+                    for (int c = 0; c < kCP; ++c) {
+                        s[c][2 * j] = fma2(keep, s[c][2 * j], mul2(kk.x, val[c]));
+                        acc[c] = fma2(s[c][2 * j], qq.x, acc[c]);
+                        s[c][2 * j + 1] = fma2(keep, s[c][2 * j + 1], mul2(kk.y, val[c]));
+                        acc[c] = fma2(s[c][2 * j + 1], qq.y, acc[c]);
                     }
                 }
 #pragma unroll
-                for (int c = 0; c < CP; ++c) {
+                for (int c = 0; c < kCP; ++c) {
                     const float2 a = parts_of(acc[c]);
-                    part[u * CP + c] = a.x + a.y;
+                    part[u * kCP + c] = a.x + a.y;
                 }
             }
-            // every exchange halves the sums a lane carries: after log2(4 CP) of them lane l holds number l mod (4 CP)
-            int o = 1;
+            // every exchange halves the sums a lane carries, while there are lanes and sums to halve: afterwards lane r
+            // holds the sums whose number is r modulo kHalved, kSums / kHalved of them
+            constexpr int kHalved = kSums < RG ? kSums : RG;
 #pragma unroll
-            for (int left = 4 * CP; left > 1; left >>= 1, o <<= 1) {
-                const bool up = lane & o;
+            for (int o = 1, left = kSums; o < kHalved; o <<= 1, left >>= 1) {
+                const bool up = r & o;
 #pragma unroll
                 for (int i = 0; i < left / 2; ++i) {
                     const float mine = up ? part[2 * i + 1] : part[2 * i], theirs = up ? part[2 * i] : part[2 * i + 1];
                     part[i] = mine + __shfl_xor_sync(0xffffffffu, theirs, o);
                 }
             }
-            float sum = part[0];
 #pragma unroll
-            for (int o2 = 4 * CP; o2 < 32; o2 <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o2);
-            if (lane < 4 * CP) {
-                const int tt = tq + lane / CP, c = wc + lane % CP;
-                if (j0 + c == dv) sum = fmaxf(fabsf(sum), sg[stage * kTT + tt].z) + 1e-6f;
-                sy[tt * cols + c] = sum;
+            for (int o = kHalved; o < RG; o <<= 1) part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
+            if (r < kHalved) {
+#pragma unroll
+                for (int i = 0; i < kSums / kHalved; ++i) {
+                    const int number = i * kHalved + r, tt = t4 + number / kCP, c = wc + number % kCP;
+                    float sum = part[i];
+                    if (j0 + c == dv) sum = fmaxf(fabsf(sum), tg[tt].z) + 1e-6f;
+                    sy[stage * kTT * cols + tt * cols + c] = sum;
+                }
             }
         }
-        shown = t0;
-        shown_n = nt;
+        __syncthreads();
     }
-    // the last tile's results: only the columns' warps still run, and they meet at a barrier of their own
-    asm volatile("bar.sync 1, %0;\n" ::"r"(threads) : "memory");
-    show();
 #pragma unroll
-    for (int c = 0; c < CP; ++c) {
+    for (int c = 0; c < kCP; ++c) {
         const int col = j0 + wc + c;
         if (col > dv) continue;
 #pragma unroll
-        for (int p = 0; p < P; ++p) {
+        for (int p = 0; p < kKR / 2; ++p) {
             const float2 e = parts_of(s[c][p]);
 #pragma unroll
             for (int x = 0; x < 2; ++x) {
-                const int i = 2 * p + x, row = (i / V) * 32 * V + lane * V + i % V;
+                const int i = 2 * p + x, row = i / 4 * 4 * RG + r * 4 + i % 4;
                 if (row >= d) continue;
                 if (col < dv) S[(size_t)row * dv + col] = x ? e.y : e.x;
                 else nn[row] = x ? e.y : e.x;
@@ -406,43 +438,49 @@ struct Args {
     float *S, *n, *m, *num; int ld_num; float* den; const int *cu_seqlens, *slots; int n_seqs, heads, d, dv; cudaStream_t stream;
 };
 
-template <typename T, int KR, int CP>
-int launch_scan(const Args& a, int warps, int vec) {
-    const int cols = warps * CP, slices = (a.dv + cols) / cols;              // dv + 1 columns
-    const size_t smem = (size_t)(2 * kTT * 32 * KR + 2 * kTT * cols + 2 * kTT * 4) * sizeof(float);
-    if (smem > 48 * 1024) {
-        const cudaError_t e = cudaFuncSetAttribute(mlstm_scan_kernel<T, KR, CP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        if (e != cudaSuccess) return (int)e;
-    }
-    return launch_chained(mlstm_scan_kernel<T, KR, CP>, dim3(a.heads * slices, a.n_seqs), dim3((warps + 1) * 32), smem, a.stream,
-                          (const T*)a.q, (const T*)a.k, (const T*)a.v, a.ld, a.gates, a.ld_gates, a.gate_bias, a.cap, a.q_scale,
-                          a.S, a.n, a.m, a.num, a.ld_num, a.den, a.cu_seqlens, a.slots, a.heads, a.d, a.dv, slices, vec);
-}
+// Measurements and tests may fix the warps of columns of a block (1, 2, 4 or 8); 0: the launcher chooses.
+static int g_warps = 0;
 
-// Measurements may fix the warps of a block (4 or 8) and the columns of a warp (2 or 4); 0: the launcher chooses.
-static int g_warps = 0, g_columns = 0;
-
-template <typename T>
-int dispatch_scan(const Args& a, int vec) {
+template <typename T, int RG>
+int launch_scan(const Args& a, int vec) {
     static int n_sm = 0;
     if (n_sm == 0) {
         int dev = 0;
         if (cudaGetDevice(&dev) != cudaSuccess || cudaDeviceGetAttribute(&n_sm, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n_sm <= 0)
             n_sm = 148;
     }
-    // wide blocks (every block stages the head's k and q again) while they still give each multiprocessor one
-    const long long columns = (long long)a.n_seqs * a.heads * a.dv;
-    int cp = columns / 32 >= 4LL * n_sm / 5 ? 4 : 2, warps = columns / (8 * cp) >= 4LL * n_sm / 5 ? 8 : 4;
-    if (g_warps == 4 || g_warps == 8) warps = g_warps;
-    if (g_columns == 2 || g_columns == 4) cp = g_columns;
-    if (a.d <= 64) return cp == 4 ? launch_scan<T, 2, 4>(a, warps, vec) : launch_scan<T, 2, 2>(a, warps, vec);
-    if (a.d <= 128) return cp == 4 ? launch_scan<T, 4, 4>(a, warps, vec) : launch_scan<T, 4, 2>(a, warps, vec);
-    if (a.d <= 256) return cp == 4 ? launch_scan<T, 8, 4>(a, warps, vec) : launch_scan<T, 8, 2>(a, warps, vec);
-    return launch_scan<T, 16, 2>(a, warps, vec);
+    constexpr int D = RG * kKR, WC = 32 / RG * kCP;
+    // as many warps a block as still give most multiprocessors a block (every block stages the head's k and q again); four
+    // where those give every multiprocessor two and the staged rows are short (measured at heads of 128 x 256: eight prompts
+    // 1,510 / 1,090 / 1,250 us at 2 / 4 / 8 warps, one prompt 246 / 277 / 424; heads of 256 x 512: eight prompts 6.1 / 4.9 /
+    // 3.7 ms, one 881 / 662 / 477 us)
+    const long long all = (long long)a.n_seqs * a.heads * ((a.dv + WC) / WC);        // warps of dv + 1 columns a head
+    int warps = kMaxWarps;
+    while (warps > 1 && all / warps < 4LL * n_sm / 5) warps /= 2;
+    if (warps == 8 && RG <= 8 && all / 4 >= 2LL * n_sm) warps = 4;
+    if (g_warps == 1 || g_warps == 2 || g_warps == 4 || g_warps == 8) warps = g_warps;
+    while (warps * WC > kMaxCols) warps /= 2;
+    const int cols = warps * WC, slices = (a.dv + cols) / cols;
+    const size_t smem = (size_t)(4 * kTT * D + 4 * kTT * cols + 2 * kTT * 4) * sizeof(float);
+    if (smem > 48 * 1024) {
+        const cudaError_t e = cudaFuncSetAttribute(mlstm_scan_kernel<T, RG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    return launch_chained(mlstm_scan_kernel<T, RG>, dim3(a.heads * slices, a.n_seqs), dim3((warps + 1) * 32 + kHelpers), smem, a.stream,
+                          (const T*)a.q, (const T*)a.k, (const T*)a.v, a.ld, a.gates, a.ld_gates, a.gate_bias, a.cap, a.q_scale,
+                          a.S, a.n, a.m, a.num, a.ld_num, a.den, a.cu_seqlens, a.slots, a.heads, a.d, a.dv, warps, slices, vec);
+}
+
+template <typename T>
+int dispatch_scan(const Args& a, int vec) {
+    if (a.d <= 64) return launch_scan<T, 4>(a, vec);
+    if (a.d <= 128) return launch_scan<T, 8>(a, vec);
+    if (a.d <= 256) return launch_scan<T, 16>(a, vec);
+    return launch_scan<T, 32>(a, vec);
 }
 }  // namespace
 
-GTG_API void gtg_mlstm_scan_shape(int warps, int columns) { g_warps = warps; g_columns = columns; }
+GTG_API void gtg_mlstm_scan_shape(int warps) { g_warps = warps; }
 
 // Most key channels a head may have.
 GTG_API int gtg_mlstm_max_key_dim() { return 512; }

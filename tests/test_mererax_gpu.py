@@ -300,8 +300,8 @@ def test_the_matrix_memory_carries_its_state_across_portions_and_slots(dtype, he
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("d,dv,n_seqs,pad", [(8, 3, 2, 0), (16, 32, 3, 0), (64, 64, 5, 0), (64, 100, 2, 3), (72, 64, 1, 0), (128, 96, 2, 0),
                                              (128, 31, 3, 8), (200, 32, 1, 0), (256, 33, 2, 0), (256, 128, 1, 0), (304, 16, 1, 0), (512, 20, 2, 0)])
-@pytest.mark.parametrize("warps,columns", [(4, 2), (8, 2), (4, 4), (8, 4)])
-def test_the_recurrence_kernel_for_every_shape_of_block(dtype, d, dv, n_seqs, pad, warps, columns):
+@pytest.mark.parametrize("warps", [1, 2, 4, 8])
+def test_the_recurrence_kernel_for_every_shape_of_block(dtype, d, dv, n_seqs, pad, warps):
     """The recurrence alone, numerators over denominators, for every block the launcher can pick: unequal sequences in
     one step, a second step that continues them, then a step of one token each; rows that allow 16-byte loads and
     rows that do not.  Both sides of the denominator's maximum occur."""
@@ -317,7 +317,7 @@ def test_the_recurrence_kernel_for_every_shape_of_block(dtype, d, dv, n_seqs, pa
     slots = torch.tensor([n_seqs - b for b in range(n_seqs)], dtype=torch.int32, device=DEV)       # not in order, slot 0 unused
     at, got = [0] * n_seqs, [[] for _ in range(n_seqs)]
     shape = build.library("mlstm").gtg_mlstm_scan_shape
-    shape(warps, columns)
+    shape(warps)
     try:
         for step_lens in lens:
             cat = lambda parts: torch.cat([p[at[b]:at[b] + step_lens[b]] for b, p in enumerate(parts)]).contiguous()
@@ -332,7 +332,7 @@ def test_the_recurrence_kernel_for_every_shape_of_block(dtype, d, dv, n_seqs, pa
                 got[b].append(o[int(cu[b]):int(cu[b + 1])])
                 at[b] += step_lens[b]
     finally:
-        shape(0, 0)
+        shape(0)
     for b in range(n_seqs):
         r, g = f64(rows[b]), f64(gates[b])
         for h in range(H):
@@ -413,6 +413,43 @@ def test_the_selective_scan_carries_its_state_across_portions_and_slots(dtype, i
         cache.advance(a, na); cache.advance(b, nb)
     close(np.concatenate(got_x), want, dtype, "first of two", loose=2.0)
     close(np.concatenate(got_y), want_y, dtype, "second of two", loose=2.0)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("states", [1, 2, 4])
+@pytest.mark.parametrize("C,N,n_seqs", [(40, 16, 3), (33, 5, 2), (64, 32, 2), (17, 30, 3), (300, 16, 1)])
+def test_the_scan_kernel_for_every_number_of_states_a_lane(dtype, states, C, N, n_seqs):
+    """The recurrence alone for every split of the states the launcher can pick: unequal sequences in one step, over several tiles
+    of tokens, a second step that continues them, then a step of one token each."""
+    rng = np.random.default_rng(C + N)
+    lens = [[1 + (37 * b + 50 * k) % 90 for b in range(n_seqs)] for k in range(2)] + [[1] * n_seqs]
+    total = [sum(l[b] for l in lens) for b in range(n_seqs)]
+    draw = lambda w: [t32(rng.standard_normal((t, w))).to(TORCH[dtype]) for t in total]
+    x, z, bc = draw(C), draw(C), draw(2 * N + 3)
+    dt = [t32(rng.standard_normal((t, C))) for t in total]
+    bias, skip, rates = t32(rng.standard_normal(C) - 1), t32(rng.standard_normal(C)), t32(-np.exp(rng.uniform(-3, 2, (C, N))))
+    state = torch.zeros(n_seqs + 1, C, N, dtype=torch.float32, device=DEV)
+    slots = torch.tensor([n_seqs - b for b in range(n_seqs)], dtype=torch.int32, device=DEV)       # not in order, slot 0 unused
+    at, got = [0] * n_seqs, [[] for _ in range(n_seqs)]
+    shape = build.library("selective").gtg_selective_scan_shape
+    shape(states)
+    try:
+        for step_lens in lens:
+            cat = lambda parts: torch.cat([p[at[b]:at[b] + step_lens[b]] for b, p in enumerate(parts)]).contiguous()
+            out = torch.empty(sum(step_lens), C, dtype=TORCH[dtype], device=DEV)
+            cu = torch.tensor(np.concatenate([[0], np.cumsum(step_lens)]), dtype=torch.int32, device=DEV)
+            ops.selective_scan(cat(x), cat(bc)[:, : 2 * N], cat(dt), bias, rates, skip, cat(z), state, out, cu, slots, n_seqs,
+                               one_token_each=max(step_lens) == 1)
+            for b in range(n_seqs):
+                got[b].append(f64(out)[int(cu[b]):int(cu[b + 1])])
+                at[b] += step_lens[b]
+    finally:
+        shape(0)
+    for b in range(n_seqs):
+        bb = f64(bc[b])
+        y = plain.selective_scan(f64(x[b]), plain.softplus(f64(dt[b]) + f64(bias)), bb[:, :N], bb[:, N:2 * N], f64(rates), f64(skip))
+        close(np.concatenate(got[b]), y * plain.silu(f64(z[b])), dtype, (C, N, states, b))
+    assert float(state[0].abs().max()) == 0.0
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
