@@ -183,7 +183,8 @@ __device__ __forceinline__ float exp2_in_order(float x) {
 // grid: (query heads, sequences, query tiles), the longest tiles first.
 // A stage of the ring: the step's keys, then its values, each as HD/64 blocks of
 // [BK tokens][64 channels] (a block holds the step's pages one after the other).
-template <int HD, bool kTest>
+// kSloped: whether `slopes` is read at all (a form of its own, so that the others keep their registers).
+template <int HD, bool kTest, bool kSloped>
 __global__ void __launch_bounds__(kThreads, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             bf16* __restrict__ out, int ldo,
@@ -230,7 +231,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     if (chunk > 0) k_min = max(k_min, (start + tile * BQ) - (start + tile * BQ) % chunk);
     const int j_lo = k_min / kPageTokens, j_hi = k_max / kPageTokens;
     const int n_steps = (j_hi - j_lo + S::kPages) / S::kPages;
-    auto first_page = [&](int i) { return j_lo + S::kPages * (slopes ? n_steps - 1 - i : i); };   // of step i
+    auto first_page = [&](int i) { return j_lo + S::kPages * (kSloped ? n_steps - 1 - i : i); };   // of step i
 
     if (threadIdx.x == 0) {
         mbar_init(q_full, 1);
@@ -324,8 +325,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int seen_from = chunk > 0 ? pos - pos % chunk : 0; // first key of this query's stretch
         const uint32_t lane_off = (uint32_t)(warp * 32) << 16;
         const float s_in = softcap > 0.f ? kLog2e : scale * kLog2e;
-        const float sl2 = slopes ? 1.0f : s_in;                  // with a slope the scores take their factor with the distance's share
-        const float slope = slopes ? slopes[h] * kLog2e : 0.f;
+        const float sl2 = kSloped ? 1.0f : s_in;                  // with a slope the scores take their factor with the distance's share
+        const float slope = kSloped ? slopes[h] * kLog2e : 0.f;
         const float cap_in = softcap > 0.f ? scale / softcap : 0.f;
         float m_run = -INFINITY, l_run = 0.f;
         uint32_t sv[BK];
@@ -356,7 +357,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
                     sv[c] = __float_as_uint(fmaf(-twice, r, softcap));
                 }
             }
-            if (slopes) {
+            if (kSloped) {
                 const float near = slope * (float)(key0 - pos);
 #pragma unroll
                 for (int c = 0; c < BK; ++c)
@@ -509,20 +510,20 @@ int make_map(CUtensorMap* map, const void* ptr, long long rows, int cols, long l
     return r == CUDA_SUCCESS ? 0 : kErrBadArgument;
 }
 
-template <int HD, bool kTest>
+template <int HD, bool kTest, bool kSloped>
 int launch(const CUtensorMap& map_q, const CUtensorMap& map_kv, bf16* out, int ldo, const int* block_table,
            int table_stride, const int* cu_seqlens, const int* slots, const int* start_pos, int B, int max_q_len,
            int n_heads, int n_kv, float scale, int window, int chunk, const float* gate, float softcap, int gate_ld,
            const float* slopes, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, kTest>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<HD, kTest, kSloped>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              Shape<HD>::kSmemBytes);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(n_heads, B, (max_q_len + BQ - 1) / BQ);
-    return launch_chained(attention_prefill_tc_kernel<HD, kTest>, grid, dim3(kThreads), (size_t)Shape<HD>::kSmemBytes, stream,
+    return launch_chained(attention_prefill_tc_kernel<HD, kTest, kSloped>, grid, dim3(kThreads), (size_t)Shape<HD>::kSmemBytes, stream,
                           map_q, map_kv, out, ldo, block_table, table_stride, cu_seqlens, slots, start_pos,
                           n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld, slopes);
 }
@@ -564,8 +565,9 @@ GTG_API int gtg_attention_prefill_tcgen05(const void* q, int ldq, int n_tokens, 
     if (st != 0) return st;
 #define GTG_ARGS map_q, map_kv, (bf16*)out, ldo, block_table, table_stride, cu_seqlens, slots, start_pos, \
                  B, max_q_len, n_heads, n_kv, scale, window, chunk, gate, softcap, gate_ld, slopes, stream
-    if (g_test_waits) return hd == 64 ? launch<64, true>(GTG_ARGS) : launch<128, true>(GTG_ARGS);
-    return hd == 64 ? launch<64, false>(GTG_ARGS) : launch<128, false>(GTG_ARGS);
+    if (g_test_waits) return hd == 64 ? launch<64, true, false>(GTG_ARGS) : launch<128, true, false>(GTG_ARGS);
+    if (slopes) return hd == 64 ? launch<64, false, true>(GTG_ARGS) : launch<128, false, true>(GTG_ARGS);
+    return hd == 64 ? launch<64, false, false>(GTG_ARGS) : launch<128, false, false>(GTG_ARGS);
 #undef GTG_ARGS
 }
 
