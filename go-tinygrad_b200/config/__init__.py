@@ -1,4 +1,5 @@
 from .llama import ConfigError, LlamaConfig, RopeScaling
+from .letanex import LetanexConfig
 from .megerax import MegeraxConfig
 from .mererax import MereraxConfig
 from .ropovik import RopovikConfig
@@ -7,6 +8,6 @@ from .zotolix import ZotolixConfig
 from .registry import (Architecture, find_architecture, read_config_json, read_model_config,
                        register_architecture, registered_architectures, unregister_architecture)
 
-__all__ = ["ConfigError", "LlamaConfig", "RopeScaling", "MegeraxConfig", "MereraxConfig", "RopovikConfig", "SenupelConfig", "ZotolixConfig", "Architecture", "find_architecture",
+__all__ = ["ConfigError", "LlamaConfig", "RopeScaling", "LetanexConfig", "MegeraxConfig", "MereraxConfig", "RopovikConfig", "SenupelConfig", "ZotolixConfig", "Architecture", "find_architecture",
            "read_config_json", "read_model_config", "register_architecture",
            "registered_architectures", "unregister_architecture"]

@@ -5,7 +5,8 @@
 // a warp takes one head (or the gates) and, all in float,
 //   * adds the biases of q, k and v;
 //   * rotates the first `rot` channels of every query and key head, channel i with
-//     i + rot/2, by the token's (cos, sin) table; the rest of a head passes;
+//     i + rot/2, by the token's (cos, sin) table; the rest of a head passes.  With `maps`
+//     > 1 a head is that many equal parts side by side and each part is rotated so;
 //   * with `unit_norm`, divides every rotated query and key head by its root mean
 //     square, x / sqrt(mean(x^2) + eps);
 //   * blends the values with those an earlier layer left for the step,
@@ -33,7 +34,7 @@ qkv_finish_rows_kernel(const float* __restrict__ sums, int ld, const float* __re
                   const int* __restrict__ block_table, int table_stride,
                   const int* __restrict__ token_seq, const int* __restrict__ slots,
                   const int* __restrict__ positions,
-                  int n_heads, int n_kv, int hd, int vd, int has_gate) {
+                  int n_heads, int n_kv, int hd, int vd, int has_gate, int maps) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float row[];
@@ -73,11 +74,13 @@ qkv_finish_rows_kernel(const float* __restrict__ sums, int ld, const float* __re
     for (int head = warp; head < n_heads + n_kv; head += n_warps) {
         float* x = row + (size_t)head * hd;
         if (cos_sin) {
-            for (int i = lane; i < rhalf; i += 32) {
+            for (int j = lane; j < maps * rhalf; j += 32) {
+                const int i = maps == 1 ? j : j % rhalf;
+                float* y = maps == 1 ? x : x + j / rhalf * (hd / maps);
                 const float2 cs = cos_sin[(size_t)n * rhalf + i];
-                const float a = x[i], b = x[i + rhalf];
-                x[i] = a * cs.x - b * cs.y;
-                x[i + rhalf] = b * cs.x + a * cs.y;
+                const float a = y[i], b = y[i + rhalf];
+                y[i] = a * cs.x - b * cs.y;
+                y[i + rhalf] = b * cs.x + a * cs.y;
             }
             __syncwarp();
         }
@@ -146,7 +149,7 @@ qkv_finish_heads_kernel(const float* __restrict__ sums, int ld, const float* __r
                   const int* __restrict__ block_table, int table_stride,
                   const int* __restrict__ token_seq, const int* __restrict__ slots,
                   const int* __restrict__ positions,
-                  int n_heads, int n_kv, int hd, int vd, int has_gate) {
+                  int n_heads, int n_kv, int hd, int vd, int has_gate, int maps) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) float staged[];          // [warp][hd]: the head a warp is turning
@@ -173,11 +176,13 @@ qkv_finish_heads_kernel(const float* __restrict__ sums, int ld, const float* __r
             __syncwarp();
             const int rhalf = rot >> 1;
             if (cos_sin) {
-                for (int i = lane; i < rhalf; i += 32) {
+                for (int j = lane; j < maps * rhalf; j += 32) {
+                    const int i = maps == 1 ? j : j % rhalf;
+                    float* y = maps == 1 ? x : x + j / rhalf * (hd / maps);
                     const float2 cs = cos_sin[(size_t)n * rhalf + i];
-                    const float a = x[i], b = x[i + rhalf];
-                    x[i] = a * cs.x - b * cs.y;
-                    x[i + rhalf] = b * cs.x + a * cs.y;
+                    const float a = y[i], b = y[i + rhalf];
+                    y[i] = a * cs.x - b * cs.y;
+                    y[i + rhalf] = b * cs.x + a * cs.y;
                 }
                 __syncwarp();
             }
@@ -526,9 +531,10 @@ GTG_API int gtg_qkv_finish(int dtype, const float* sums, int ld, const float* bi
                            int unit_norm, float eps, const float* v_first, float* v_keep, float lambda,
                            void* q_out, int ldq, float* gate_out, void* kc, void* vc, long long page_stride,
                            const int* block_table, int table_stride, const int* token_seq, const int* slots,
-                           const int* positions, int N, int n_heads, int n_kv, int hd, int vd, cudaStream_t stream) {
+                           const int* positions, int N, int n_heads, int n_kv, int hd, int vd, int maps, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (n_heads <= 0 || n_kv <= 0 || hd <= 0 || vd <= 0 || rot < 0 || (rot & 1) || rot > hd) return kErrBadArgument;
+    if (n_heads <= 0 || n_kv < 0 || hd <= 0 || vd <= 0 || maps < 1 || hd % maps || rot < 0 || (rot & 1) || rot > hd / maps) return kErrBadArgument;
+    if (n_kv == 0 && (kc || v_first || v_keep)) return kErrBadArgument;
     if ((cos_sin != nullptr) != (rot > 0) || (kc == nullptr) != (vc == nullptr)) return kErrBadArgument;
     const int has_gate = gate_out != nullptr;
     const int width = n_heads * hd + n_kv * (hd + vd) + (has_gate ? n_heads : 0);
@@ -551,7 +557,7 @@ GTG_API int gtg_qkv_finish(int dtype, const float* sums, int ld, const float* bi
         return launch_chained(kernel, grid, dim3(kFinishWarps * 32), smem, stream, sums, ld, bias, (const float2*)cos_sin, rot, \
                               unit_norm, eps, v_first, v_keep, lambda, (T*)q_out, ldq, gate_out, (T*)kc, (T*)vc,    \
                               page_stride, block_table, table_stride, token_seq, slots, positions, n_heads, n_kv,  \
-                              hd, vd, has_gate);                                                                   \
+                              hd, vd, has_gate, maps);                                                                   \
     } while (0)
     if (dtype == 0) GTG_FINISH(float);
     if (dtype == 1) GTG_FINISH(bf16);

@@ -86,14 +86,27 @@ constexpr int kActivations = 3;
 // Epilogue code 1 is the gated product over interleaved rows, silu(gate) * up; from this value on it is
 // the same with activation (code - kEpiGated) on the gate in silu's place.
 constexpr int kEpiGated = 32;
+// Codes from kEpiClamped on are the clamped gated product: the code is the bit pattern of a positive float,
+// the limit L, and with g = min(gate, L) and u = up between -L and L the result is g sigmoid(1.702 g) (u + 1).
+// (The smallest normal float's bits lie far above every other code.)
+constexpr int kEpiClamped = 0x00800000;
+__host__ __device__ __forceinline__ bool epi_is_clamped(int code) { return code >= kEpiClamped; }
 __host__ __device__ __forceinline__ bool epi_is_gated(int code) {
-    return code == 1 || (code >= kEpiGated && code < kEpiGated + kActivations);
+    return code == 1 || (code >= kEpiGated && code < kEpiGated + kActivations) || epi_is_clamped(code);
 }
 __host__ __device__ __forceinline__ bool epi_is_activation(int code) {
     return code >= kEpiActivation && code < kEpiActivation + kActivations;
 }
-__device__ __forceinline__ float gate_activate(float g, int code) {
-    return code == 1 ? g / (1.0f + expf(-g)) : activate(g, code - kEpiGated);
+__device__ __forceinline__ float clamped_gate(float g, float u, float limit) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+// A gated product's result from its two float sums, for every gated epilogue code.
+__device__ __forceinline__ float gated_value(float g, float u, int code) {
+    if (code == 1) return g / (1.0f + expf(-g)) * u;
+    if (epi_is_clamped(code)) return clamped_gate(g, u, __int_as_float(code));
+    return activate(g, code - kEpiGated) * u;
 }
 
 static inline int launch_status() {

@@ -516,6 +516,47 @@ head_norm_gate_vec_kernel(const float* __restrict__ y, int ld_y, const G* __rest
     }
 }
 
+// The same for wide heads (a row normed as one head): a block of 256 threads per (token, head), KV pieces of four
+// channels a thread (dv <= 1024 KV).
+template <typename T, typename G, int KV>
+__global__ void __launch_bounds__(256)
+head_norm_gate_block_kernel(const float* __restrict__ y, int ld_y, const G* __restrict__ gate, int ld_gate,
+                            const float* __restrict__ weight, int w_step, float eps, const float* __restrict__ den,
+                            T* __restrict__ out, int ld_out, int n_heads, int dv) {
+    chain_release();
+    chain_wait();
+    __shared__ float scratch[33];
+    const size_t n = blockIdx.x / n_heads;
+    const int h = blockIdx.x % n_heads;
+    const float* src = y + n * ld_y + (size_t)h * dv;
+    const G* gt = gate + n * ld_gate + (size_t)h * dv;
+    const float* w = weight + (size_t)h * w_step;
+    float4 v[KV], g[KV];
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        const int c = ((int)threadIdx.x + 256 * k) * 4;
+        v[k] = c < dv ? load_four(src + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        g[k] = c < dv ? load_four(gt + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float part = den ? 1.0f / den[blockIdx.x] : 1.0f;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        v[k].x *= part; v[k].y *= part; v[k].z *= part; v[k].w *= part;
+        ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
+    T* dst = out + n * ld_out + (size_t)h * dv;
+#pragma unroll
+    for (int k = 0; k < KV; ++k) {
+        const int c = ((int)threadIdx.x + 256 * k) * 4;
+        if (c >= dv) continue;
+        const float4 ww = load_four(w + c);
+        store_four(dst + c, make_float4(v[k].x * inv * ww.x / (1.0f + expf(-g[k].x)), v[k].y * inv * ww.y / (1.0f + expf(-g[k].y)),
+                                        v[k].z * inv * ww.z / (1.0f + expf(-g[k].z)), v[k].w * inv * ww.w / (1.0f + expf(-g[k].w))));
+    }
+}
+
 template <typename T, typename G>
 static int launch_head_norm_gate(const float* y, int ld_y, const void* gate, int ld_gate, const float* weight, int w_step, float eps,
                                  const float* den, void* out, int ld_out, long long items, int n_heads, int dv, cudaStream_t stream) {
@@ -528,6 +569,13 @@ static int launch_head_norm_gate(const float* y, int ld_y, const void* gate, int
     if (fours && dv <= 128) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 1>));
     if (fours && dv <= 256) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 2>));
     if (fours && dv <= 512) GTG_HEAD_NORM((head_norm_gate_vec_kernel<T, G, 4>));
+#define GTG_HEAD_NORM_BLOCK(KV)                                                                                      \
+    return launch_chained(head_norm_gate_block_kernel<T, G, KV>, dim3((unsigned)items), dim3(256), 0, stream, y, ld_y, (const G*)gate, \
+                          ld_gate, weight, w_step, eps, den, (T*)out, ld_out, n_heads, dv)
+    if (fours && dv <= 1024 && items <= 0x7fffffffLL) GTG_HEAD_NORM_BLOCK(1);
+    if (fours && dv <= 2048 && items <= 0x7fffffffLL) GTG_HEAD_NORM_BLOCK(2);
+    if (fours && dv <= 8192 && items <= 0x7fffffffLL) GTG_HEAD_NORM_BLOCK(8);
+#undef GTG_HEAD_NORM_BLOCK
     GTG_HEAD_NORM((head_norm_gate_kernel<T, G>));
 #undef GTG_HEAD_NORM
 }

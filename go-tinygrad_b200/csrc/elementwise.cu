@@ -189,7 +189,8 @@ GTG_API int gtg_add_rmsnorm(int dtype, float* residual, const void* pending, con
 
 // ------------------------------------------------------------------ SwiGLU
 // out[m,i] = act(gu[m,i]) * gu[m,I+i]; act is silu, g / (1 + exp(-g))
-// (backends/simd/vec.go:52-59), or another of the pointwise activations (`kind`).
+// (backends/simd/vec.go:52-59), or another of the pointwise activations (`kind`; from
+// kEpiClamped on it is the clamped gated product's code instead).
 // `gu` holds the gate columns then the up columns.
 template <typename T>
 __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int ldo, int M, int I, int kind) {
@@ -202,15 +203,14 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
         const int i = (int)(idx - m * I);
         const float g = to_f32<T>(gu[m * 2 * I + i]);
         const float u = to_f32<T>(gu[m * 2 * I + I + i]);
-        const float s = kind == 2 ? g / (1.0f + expf(-g)) : activate(g, kind);
-        out[m * ldo + i] = from_f32<T>(s * u);
+        out[m * ldo + i] = from_f32<T>(kind == 2 ? g / (1.0f + expf(-g)) * u : epi_is_clamped(kind) ? gated_value(g, u, kind) : activate(g, kind) * u);
     }
 }
 
 GTG_API int gtg_swiglu(int dtype, const void* gu, void* out, int ldo, int M, int I, int kind, cudaStream_t stream) {
     int st = 0;
     if (M <= 0 || I <= 0) return 0;
-    if (kind < 0 || kind >= kActivations || ldo < I) return kErrBadArgument;
+    if (kind < 0 || (kind >= kActivations && !epi_is_clamped(kind)) || ldo < I) return kErrBadArgument;
     const size_t total = (size_t)M * I;
     int blocks = (int)((total + 255) / 256);
     if (blocks > 148 * 16) blocks = 148 * 16;
@@ -604,6 +604,179 @@ GTG_API int gtg_add_layernorm(int dtype, float* residual, const void* pending, c
     return kErrBadArgument;
 }
 
+// ----------------------------- a normed update joins the hidden state, which is normed again
+// x = residual[r,:] + LN(update[r,:]; weight_u);  out[i,:] = LN(x; weight) + bias, LN(x; w) =
+// (x - mean) / sqrt(var + eps) * w, var the mean of the squared deviations: the arrangement in which a
+// sublayer stands between two norms, the second of which meets the first of the next sublayer here.
+// U is the update's type (float from a product that kept its sums).  Rows as in add_rmsnorm: with `rows`
+// nothing is written back.  Everything in float.
+template <typename U, typename T>
+__global__ void layernorm_add_layernorm_kernel(float* __restrict__ residual, const U* __restrict__ update,
+                                               const float* __restrict__ weight_u, float eps_u,
+                                               const float* __restrict__ weight, const float* __restrict__ bias, float eps,
+                                               T* __restrict__ out, const int* __restrict__ rows, int H) {
+    chain_release();
+    chain_wait();
+    extern __shared__ float smem[];
+    float* row = smem;          // H floats
+    float* scratch = smem + H;  // 33 floats
+    const int i_out = blockIdx.x;
+    const int r = rows ? rows[i_out] : i_out;
+    float* res = residual + (size_t)r * H;
+    const U* up = update + (size_t)r * H;
+    auto deviation = [&](float sum, float& mean) {          // of the row in shared memory: its mean and its variance
+        mean = block_sum(sum, scratch) / (float)H;
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) {
+            const float d = row[i] - mean;
+            ss += d * d;
+        }
+        return block_sum(ss, scratch) / (float)H;
+    };
+    float sum = 0.f, mean;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float u = to_f32<U>(up[i]);
+        row[i] = u;
+        sum += u;
+    }
+    float s = 1.0f / sqrtf(deviation(sum, mean) + eps_u);
+    sum = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {
+        const float x = res[i] + (row[i] - mean) * s * weight_u[i];
+        if (!rows) res[i] = x;
+        row[i] = x;
+        sum += x;
+    }
+    s = 1.0f / sqrtf(deviation(sum, mean) + eps);
+    T* o = out + (size_t)i_out * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+        o[i] = from_f32<T>((row[i] - mean) * s * weight[i] + (bias ? bias[i] : 0.f));
+}
+
+// Sum over the block with one barrier: every warp leaves its sum in `part` and every thread adds them up.
+// Sums that follow one another use different `part`s (32 floats each).
+__device__ __forceinline__ float block_sum_once(float v, float* part) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+    __syncthreads();
+    const int n = blockDim.x >> 5;
+    float t = 0.f;
+    for (int w = 0; w < n; ++w) t += part[w];
+    return t;
+}
+
+__device__ __forceinline__ void load_eight(const float* p, float* x) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+}
+__device__ __forceinline__ void load_eight(const bf16* p, float* x) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        const float2 f = __bfloat1622float2(h[j]);
+        x[2 * j] = f.x;
+        x[2 * j + 1] = f.y;
+    }
+}
+
+// The same for bfloat16 rows whose width is a multiple of 8 and at most 8192: every thread owns 8
+// consecutive channels, kept in registers from the first read to the last write.
+template <typename U>
+__global__ void __launch_bounds__(1024)
+layernorm_add_layernorm_vec_kernel(float* __restrict__ residual, const U* __restrict__ update,
+                                   const float* __restrict__ weight_u, float eps_u,
+                                   const float* __restrict__ weight, const float* __restrict__ bias, float eps,
+                                   bf16* __restrict__ out, const int* __restrict__ rows, int H) {
+    chain_release();
+    chain_wait();        // before every load: one through a restricted pointer to const may be moved over a later wait
+    __shared__ float part[4][32];
+    const int c = threadIdx.x * 8;
+    const bool active = c < H;
+    float wu[8], w[8], b[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (active) {
+        load_eight(weight_u + c, wu);
+        load_eight(weight + c, w);
+        if (bias) load_eight(bias + c, b);
+    }
+    const int i_out = blockIdx.x;
+    const int r = rows ? rows[i_out] : i_out;
+    float u[8], x[8];
+    float* rp = residual + (size_t)r * H + c;
+    float sum = 0.f;
+    if (active) {
+        load_eight(update + (size_t)r * H + c, u);
+        load_eight(rp, x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sum += u[j];
+    }
+    float mean = block_sum_once(sum, part[0]) / (float)H;
+    float ss = 0.f;
+    if (active) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { u[j] -= mean; ss += u[j] * u[j]; }
+    }
+    float s = 1.0f / sqrtf(block_sum_once(ss, part[1]) / (float)H + eps_u);
+    sum = 0.f;
+    if (active) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { x[j] += u[j] * s * wu[j]; sum += x[j]; }
+        if (!rows) {
+            reinterpret_cast<float4*>(rp)[0] = make_float4(x[0], x[1], x[2], x[3]);
+            reinterpret_cast<float4*>(rp)[1] = make_float4(x[4], x[5], x[6], x[7]);
+        }
+    }
+    mean = block_sum_once(sum, part[2]) / (float)H;
+    ss = 0.f;
+    if (active) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) { x[j] -= mean; ss += x[j] * x[j]; }
+    }
+    s = 1.0f / sqrtf(block_sum_once(ss, part[3]) / (float)H + eps);
+    if (active) {
+        uint4 o;
+        __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            oh[j] = __floats2bfloat162_rn(x[2 * j] * s * w[2 * j] + b[2 * j], x[2 * j + 1] * s * w[2 * j + 1] + b[2 * j + 1]);
+        *reinterpret_cast<uint4*>(out + (size_t)i_out * H + c) = o;
+    }
+}
+
+GTG_API int gtg_layernorm_add_layernorm(int dtype, int update_f32, float* residual, const void* update, const float* weight_u,
+                                        float eps_u, const float* weight, const float* bias, float eps, void* out,
+                                        const int* rows, int R, int H, cudaStream_t stream) {
+    if (R <= 0) return 0;
+    if (H <= 0 || !update || !weight_u || !weight) return kErrBadArgument;
+    if (dtype == 1 && H % 8 == 0 && H <= 8192 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
+        ((uintptr_t)weight % 16) == 0 && ((uintptr_t)weight_u % 16) == 0 && ((uintptr_t)bias % 16) == 0 && ((uintptr_t)update % 16) == 0) {
+        const int t = ((H / 8) + 31) / 32 * 32;
+        if (update_f32)
+            return launch_chained(layernorm_add_layernorm_vec_kernel<float>, dim3(R), dim3(t), 0, stream, residual, (const float*)update,
+                                  weight_u, eps_u, weight, bias, eps, (bf16*)out, rows, H);
+        return launch_chained(layernorm_add_layernorm_vec_kernel<bf16>, dim3(R), dim3(t), 0, stream, residual, (const bf16*)update,
+                              weight_u, eps_u, weight, bias, eps, (bf16*)out, rows, H);
+    }
+    int threads = 32;
+    while (threads < 1024 && threads * 4 < H) threads *= 2;
+    const size_t smem = (size_t)(H + 33) * sizeof(float);
+    if (smem > 200 * 1024) return kErrUnsupported;
+#define GTG_NORM_ADD_NORM(U, T)                                                                                  \
+    do {                                                                                                         \
+        if (smem > 48 * 1024) {                                                                                  \
+            const cudaError_t e = cudaFuncSetAttribute(layernorm_add_layernorm_kernel<U, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            if (e != cudaSuccess) return (int)e;                                                                 \
+        }                                                                                                        \
+        return launch_chained(layernorm_add_layernorm_kernel<U, T>, dim3(R), dim3(threads), smem, stream, residual, (const U*)update, \
+                              weight_u, eps_u, weight, bias, eps, (T*)out, rows, H);                             \
+    } while (0)
+    if (dtype == 0) GTG_NORM_ADD_NORM(float, float);
+    if (dtype == 1 && update_f32) GTG_NORM_ADD_NORM(float, bf16);
+    if (dtype == 1) GTG_NORM_ADD_NORM(bf16, bf16);
+#undef GTG_NORM_ADD_NORM
+    return kErrBadArgument;
+}
+
 // ------------------------------------------------------ pointwise activations
 // x <- f(x) in place, evaluated in float.  kind 0: relu(x)^2; 1: gelu in its tanh
 // form, 0.5 x (1 + tanh(sqrt(2/pi) (x + 0.044715 x^3))); 2: silu, x / (1 + exp(-x)).
@@ -842,10 +1015,11 @@ GTG_API int gtg_round_rows(int dtype, const float* x, void* out, long long total
 }
 
 // ---- biases ------------------------------------------------------------------------
-// out[m,i] = silu(gu[m,i] + bg[i]) * (gu[m,I+i] + bu[i]) from a product's float sums.
+// out[m,i] = silu(gu[m,i] + bg[i]) * (gu[m,I+i] + bu[i]) from a product's float sums; with another gated
+// epilogue's `code` than 1, that product of the two in silu's place.
 template <typename T>
 __global__ void swiglu_bias_kernel(const float* __restrict__ gu, const float* __restrict__ bg,
-                                   const float* __restrict__ bu, T* __restrict__ out, int ldo, int M, int I) {
+                                   const float* __restrict__ bu, T* __restrict__ out, int ldo, int M, int I, int code) {
     chain_release();
     chain_wait();
     const size_t total = (size_t)M * I;
@@ -854,17 +1028,18 @@ __global__ void swiglu_bias_kernel(const float* __restrict__ gu, const float* __
         const int i = (int)(idx % I);
         const float g = gu[m * 2 * I + i] + (bg ? bg[i] : 0.f);
         const float u = gu[m * 2 * I + I + i] + (bu ? bu[i] : 0.f);
-        out[m * ldo + i] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+        out[m * ldo + i] = from_f32<T>(gated_value(g, u, code));
     }
 }
 
 GTG_API int gtg_swiglu_bias(int dtype, const float* gu, const float* bg, const float* bu, void* out, int ldo,
-                            int M, int I, cudaStream_t stream) {
+                            int M, int I, int code, cudaStream_t stream) {
     if (M <= 0 || I <= 0) return 0;
+    if (!epi_is_gated(code)) return kErrBadArgument;
     const size_t total = (size_t)M * I;
     const unsigned blocks = (unsigned)((total + 255) / 256 > 8192 ? 8192 : (total + 255) / 256);
-    if (dtype == 0) return launch_chained(swiglu_bias_kernel<float>, dim3(blocks), dim3(256), 0, stream, gu, bg, bu, (float*)out, ldo, M, I);
-    if (dtype == 1) return launch_chained(swiglu_bias_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, gu, bg, bu, (bf16*)out, ldo, M, I);
+    if (dtype == 0) return launch_chained(swiglu_bias_kernel<float>, dim3(blocks), dim3(256), 0, stream, gu, bg, bu, (float*)out, ldo, M, I, code);
+    if (dtype == 1) return launch_chained(swiglu_bias_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, gu, bg, bu, (bf16*)out, ldo, M, I, code);
     return kErrBadArgument;
 }
 

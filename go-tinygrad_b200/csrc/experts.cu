@@ -6,12 +6,15 @@
 //   route    z = R x + b in float; the `top` largest z (ties: the lower index)
 //            are the token's experts, their weights softmax over those z alone
 //            (scoring 0) or each chosen expert's own sigmoid(z), not renormalised
-//            (scoring 1; the largest sigmoid is the largest z).
+//            (scoring 1; the largest sigmoid is the largest z).  Scoring 2: s = softmax(z) over
+//            all outputs, the largest s + correction are chosen, and the weights are the
+//            chosen s over their sum (+ 1e-20) times weight_scale.
 //   arrange  item i = (token i / top, its (i % top)-th expert).  Items of one
 //            expert get consecutive rows, every expert's stretch padded to whole
 //            tiles of `tile` rows, so that a tile of rows has one expert:
 //            row_item[row] = item or -1, item_row[item] = row, tile_expert[tile]
-//            = expert or -1 past the last tile.  Which of an expert's rows an
+//            = expert or -1 past the last tile.  A choice of E or more stands for no expert
+//            (an identity): its item has no row, item_row[item] = -1.  Which of an expert's rows an
 //            item gets is arbitrary; no result depends on it, since every row is
 //            computed by itself.
 //   product  C[row,:] = A[source(row),:] . W[expert(row)]^T, tiles of 64 rows,
@@ -21,7 +24,8 @@
 //            weights, G[row,:] = weight[item] * x[token,:], the product in float and
 //            rounded once: a mixture whose weights scale an expert's input.
 //   combine  out[t,:] = sum_k weight[t,k] * Y[item_row[t*top+k],:], k in order
-//            (weights null: the plain sum).
+//            (weights null: the plain sum); an item without a row stands for the token's own
+//            input x[t,:]; with `base`, base[t,:] is added last.
 #include "common.cuh"
 #include <math.h>
 
@@ -43,14 +47,15 @@ __device__ __forceinline__ float4 four_channels(const bf16* p) {
 template <typename T, int TB>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ router, const float* __restrict__ bias,
-                 int* __restrict__ chosen, float* __restrict__ weights, int N, int H, int E, int top, int scoring) {
+                 int* __restrict__ chosen, float* __restrict__ weights, int N, int H, int E, int top, int scoring,
+                 const float* __restrict__ correction, float weight_scale) {
     chain_release();
     chain_wait();
     extern __shared__ __align__(16) unsigned char route_smem[];
     constexpr int kPer16 = 16 / (int)sizeof(T);          // channels in 16 bytes
     const int Hp = (H + kPer16 - 1) / kPer16 * kPer16;   // a staged row, whole 16 bytes
     T* xs = reinterpret_cast<T*>(route_smem);            // [TB][Hp]
-    float* zs = reinterpret_cast<float*>(route_smem + (size_t)TB * Hp * sizeof(T));   // [TB][2 E]: logits, then the chosen scores
+    float* zs = reinterpret_cast<float*>(route_smem + (size_t)TB * Hp * sizeof(T));   // [TB][2 E]: logits or choice scores, then scores
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n0 = blockIdx.x * TB;
     const int nt = min(TB, N - n0);
@@ -102,29 +107,57 @@ moe_route_kernel(const T* __restrict__ x, int ldx, const float* __restrict__ rou
         }
     }
     __syncthreads();
-    if (threadIdx.x < nt) {
-        const int n = n0 + threadIdx.x;
-        float* z = zs + threadIdx.x * 2 * E;
-        float* kept = z + E;
-        // top <= E rounds of a first-maximum search; a chosen logit becomes NaN, which no comparison picks again
+    if (warp < nt) {
+        // a warp a token: rounds of a first-maximum search over the lanes; what was chosen becomes NaN, which no
+        // comparison picks again
+        const int n = n0 + warp;
+        float* z = zs + warp * 2 * E;
+        float* score = z + E;                               // scoring 2: the softmax over all outputs
+        if (scoring == 2) {
+            float mx = -INFINITY, sum = 0.f;
+            for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+            mx = warp_max(mx);
+            for (int e = lane; e < E; e += 32) {
+                score[e] = expf(z[e] - mx);
+                sum += score[e];
+            }
+            sum = warp_sum(sum);
+            for (int e = lane; e < E; e += 32) {
+                score[e] /= sum;
+                z[e] = score[e] + (correction ? correction[e] : 0.f);
+            }
+            __syncwarp();
+        }
         float best0 = 0.f, total = 0.f;
         for (int k = 0; k < top; ++k) {
-            int arg = -1;
+            int arg = E;
             float best = -INFINITY;
-            for (int e = 0; e < E; ++e) {
+            for (int e = lane; e < E; e += 32) {
                 const float v = z[e];
                 if (v != v) continue;                       // chosen in an earlier round
-                if (arg < 0 || v > best) { best = v; arg = e; }
+                if (arg == E || v > best) { best = v; arg = e; }
             }
-            z[arg] = __int_as_float(0x7fc00000);
-            if (k == 0) best0 = best;
-            chosen[(size_t)n * top + k] = arg;
-            const float p = scoring == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - best0);
-            kept[k] = p;
-            total += p;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+                if (oa < E && (arg == E || ob > best || (ob == best && oa < arg))) { best = ob; arg = oa; }
+            }
+            if (arg == E) arg = 0;                          // only NaN is left: any output will do
+            if (lane == 0) {
+                z[arg] = __int_as_float(0x7fc00000);
+                if (k == 0) best0 = best;
+                chosen[(size_t)n * top + k] = arg;
+                const float p = scoring == 2 ? score[arg] : scoring == 1 ? 1.0f / (1.0f + expf(-best)) : expf(best - best0);
+                weights[(size_t)n * top + k] = p;
+                total += p;
+            }
+            __syncwarp();
         }
-        const float inv = scoring == 1 ? 1.0f : 1.0f / total;
-        for (int k = 0; k < top; ++k) weights[(size_t)n * top + k] = kept[k] * inv;
+        if (lane == 0 && scoring != 1) {
+            const float inv = scoring == 2 ? weight_scale / (total + 1e-20f) : 1.0f / total;
+            for (int k = 0; k < top; ++k) weights[(size_t)n * top + k] *= inv;
+        }
     }
 }
 
@@ -140,7 +173,7 @@ moe_arrange_kernel(const int* __restrict__ chosen, int n_items, int E, int tile,
     int* cursor = ism + 2 * E;   // [E]
     for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = cursor[e] = 0;
     __syncthreads();
-    for (int i = threadIdx.x; i < n_items; i += blockDim.x) atomicAdd(&count[chosen[i]], 1);
+    for (int i = threadIdx.x; i < n_items; i += blockDim.x) if (chosen[i] < E) atomicAdd(&count[chosen[i]], 1);
     __syncthreads();
     if (threadIdx.x == 0) {
         int t = 0;
@@ -156,6 +189,7 @@ moe_arrange_kernel(const int* __restrict__ chosen, int n_items, int E, int tile,
     __syncthreads();
     for (int i = threadIdx.x; i < n_items; i += blockDim.x) {
         const int e = chosen[i];
+        if (e >= E) { item_row[i] = -1; continue; }
         const int row = first[e] + atomicAdd(&cursor[e], 1);
         row_item[row] = i;
         item_row[i] = row;
@@ -284,25 +318,31 @@ __global__ void moe_gather_scaled_wide_kernel(const bf16* __restrict__ x, int ld
 }
 
 // ---- combine ----------------------------------------------------------------------
-template <typename T>
+template <typename T, typename X>
 __global__ void moe_combine_kernel(const float* __restrict__ y, int ldy, const int* __restrict__ item_row,
-                                   const float* __restrict__ weights, T* __restrict__ out, int H, int top) {
+                                   const float* __restrict__ weights, T* __restrict__ out, int H, int top,
+                                   const X* __restrict__ x, int ldx, const float* __restrict__ base) {
     chain_release();
     chain_wait();
     const int t = blockIdx.x;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float s = 0.f;
-        for (int k = 0; k < top; ++k)
-            s = fmaf(weights ? weights[(size_t)t * top + k] : 1.0f, y[(size_t)item_row[(size_t)t * top + k] * ldy + i], s);
+        for (int k = 0; k < top; ++k) {
+            const int row = item_row[(size_t)t * top + k];
+            const float v = row >= 0 ? y[(size_t)row * ldy + i] : to_f32<X>(x[(size_t)t * ldx + i]);
+            s = fmaf(weights ? weights[(size_t)t * top + k] : 1.0f, v, s);
+        }
+        if (base) s += base[(size_t)t * H + i];
         out[(size_t)t * H + i] = from_f32<T>(s);
     }
 }
 }  // namespace
 
 GTG_API int gtg_moe_route(int dtype, const void* x, int ldx, const float* router, const float* bias, int* chosen,
-                          float* weights, int N, int H, int E, int top, int scoring, cudaStream_t stream) {
+                          float* weights, int N, int H, int E, int top, int scoring, const float* correction,
+                          float weight_scale, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (E <= 0 || top <= 0 || top > E || H <= 0 || scoring < 0 || scoring > 1) return kErrBadArgument;
+    if (E <= 0 || top <= 0 || top > E || H <= 0 || scoring < 0 || scoring > 2 || (correction && scoring != 2)) return kErrBadArgument;
     // many tokens: four share a block, so that the router is read a quarter as often
     const size_t elem = dtype == 0 ? 4 : 2;
     const size_t row = ((size_t)H * elem + 15) / 16 * 16;
@@ -318,7 +358,7 @@ GTG_API int gtg_moe_route(int dtype, const void* x, int ldx, const float* router
             if (e != cudaSuccess) return (int)e;                                                                   \
         }                                                                                                          \
         return launch_chained(kernel, grid, dim3(256), smem, stream, (const T*)x, ldx, router, bias, chosen, weights, \
-                              N, H, E, top, scoring);                                                              \
+                              N, H, E, top, scoring, correction, weight_scale);                                                              \
     } while (0)
     if (dtype == 0) { if (tb == 4) GTG_ROUTE(float, 4); else GTG_ROUTE(float, 1); }
     if (dtype == 1) { if (tb == 4) GTG_ROUTE(bf16, 4); else GTG_ROUTE(bf16, 1); }
@@ -384,11 +424,15 @@ GTG_API int gtg_moe_gather_scaled(int dtype, const void* x, int ldx, const int* 
     return kErrBadArgument;
 }
 
+// dtype: of out, and of x where the arrangement leaves items without a row (null where it leaves none).
 GTG_API int gtg_moe_combine(int dtype, const float* y, int ldy, const int* item_row, const float* weights, void* out,
-                            int N, int H, int top, cudaStream_t stream) {
+                            int N, int H, int top, const void* x, int ldx, int x_bf16, const float* base, cudaStream_t stream) {
     if (N <= 0) return 0;
-    if (H <= 0 || top <= 0) return kErrBadArgument;
-    if (dtype == 0) return launch_chained(moe_combine_kernel<float>, dim3(N), dim3(256), 0, stream, y, ldy, item_row, weights, (float*)out, H, top);
-    if (dtype == 1) return launch_chained(moe_combine_kernel<bf16>, dim3(N), dim3(256), 0, stream, y, ldy, item_row, weights, (bf16*)out, H, top);
+    if (H <= 0 || top <= 0 || (x && ldx < H)) return kErrBadArgument;
+#define GTG_COMBINE(T, X) return launch_chained(moe_combine_kernel<T, X>, dim3(N), dim3(256), 0, stream, y, ldy, item_row, weights, (T*)out, H, top, (const X*)x, ldx, base)
+    if (dtype == 0 && !x_bf16) GTG_COMBINE(float, float);
+    if (dtype == 0) GTG_COMBINE(float, bf16);
+    if (dtype == 1) GTG_COMBINE(bf16, bf16);
+#undef GTG_COMBINE
     return kErrBadArgument;
 }

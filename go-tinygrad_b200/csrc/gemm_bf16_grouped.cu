@@ -175,14 +175,14 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, long long batch_a, const
             const int r = wm * (BM / 2) + i * 16 + g + half * 8;
             if (src[r] < 0) continue;
             const size_t m = (size_t)(m0 + r);
-            if (epilogue == 1) {
+            if (epi_is_gated(epilogue)) {
 #pragma unroll
                 for (int j = 0; j < 4; j += 2) {
                     const int n = n0 + wn * 32 + j * 8;              // a block of 8 gate rows, then their 8 up rows
                     if (pairs && n + 16 <= N) {
                         const float g0 = acc[i][j][half * 2], g1 = acc[i][j][half * 2 + 1];
-                        put2<OutT>(C + m * ldc + n / 2 + t * 2, g0 / (1.0f + expf(-g0)) * acc[i][j + 1][half * 2],
-                                   g1 / (1.0f + expf(-g1)) * acc[i][j + 1][half * 2 + 1]);
+                        put2<OutT>(C + m * ldc + n / 2 + t * 2, gated_value(g0, acc[i][j + 1][half * 2], epilogue),
+                                   gated_value(g1, acc[i][j + 1][half * 2 + 1], epilogue));
                         continue;
                     }
 #pragma unroll
@@ -190,7 +190,7 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, long long batch_a, const
                         const int col = n / 2 + t * 2 + e;
                         if (n + 8 + t * 2 + e < N) {
                             const float gate = acc[i][j][half * 2 + e], up = acc[i][j + 1][half * 2 + e];
-                            put<OutT>(C + m * ldc + col, gate / (1.0f + expf(-gate)) * up);
+                            put<OutT>(C + m * ldc + col, gated_value(gate, up, epilogue));
                         }
                     }
                 }
@@ -200,7 +200,7 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, long long batch_a, const
                     const int n2 = n0 + wn * 32 + j * 8 + t * 2;
                     if (pairs && n2 + 1 < N) {
                         float v0 = acc[i][j][half * 2], v1 = acc[i][j][half * 2 + 1];
-                        if (epilogue >= kEpiActivation) { v0 = activate(v0, epilogue - kEpiActivation); v1 = activate(v1, epilogue - kEpiActivation); }
+                        if (epi_is_activation(epilogue)) { v0 = activate(v0, epilogue - kEpiActivation); v1 = activate(v1, epilogue - kEpiActivation); }
                         if (epilogue == 2) {
                             const float2 gg = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(G + m * ldg + n2));
                             v0 *= 1.0f / (1.0f + expf(-gg.x));
@@ -214,7 +214,7 @@ grouped_mma_kernel(const bf16* __restrict__ A, int lda, long long batch_a, const
                         const int n = n0 + wn * 32 + j * 8 + t * 2 + e;
                         if (n >= N) continue;
                         float v = acc[i][j][half * 2 + e];
-                        if (epilogue >= kEpiActivation) v = activate(v, epilogue - kEpiActivation);
+                        if (epi_is_activation(epilogue)) v = activate(v, epilogue - kEpiActivation);
                         if (epilogue == 2) v *= 1.0f / (1.0f + expf(-__bfloat162float(G[m * ldg + n])));
                         put<OutT>(C + m * ldc + n, v);
                     }
@@ -250,10 +250,10 @@ GTG_API int gtg_gemm_bf16_grouped(const void* A, int lda, long long batch_a, con
                                   long long batch_c, int out_f32, int batch, int M, int N, int K, int tile_rows,
                                   int epilogue, const void* G, int ldg, long long batch_g, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || batch <= 0) return 0;
-    if (K <= 0 || lda < K || ldw < K || epilogue < 0 || (epilogue > 2 && !(epilogue >= kEpiActivation && epilogue < kEpiActivation + kActivations)) ||
+    if (K <= 0 || lda < K || ldw < K || !(epilogue == 0 || epilogue == 2 || epi_is_gated(epilogue) || epi_is_activation(epilogue)) ||
         (epilogue == 2 && !G)) return kErrBadArgument;
     if (K % 8 || lda % 8 || ldw % 8 || batch_a % 8 || batch_w % 8 || ((uintptr_t)A % 16) || ((uintptr_t)W % 16)) return kErrUnsupported;
-    if (epilogue == 1 && N % 16) return kErrUnsupported;
+    if (epi_is_gated(epilogue) && N % 16) return kErrUnsupported;
     if (tile_expert && batch != 1) return kErrBadArgument;
 #define GTG_GROUPED(BM, BK, ST, T)                                                                                  \
     return launch<BM, BK, ST, T>((const bf16*)A, lda, batch_a, row_item, item_div, (const bf16*)W, ldw, batch_w, tile_expert, \

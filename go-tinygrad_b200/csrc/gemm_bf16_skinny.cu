@@ -97,7 +97,7 @@ __device__ __forceinline__ void store_feature(OutT* C, int ldc, int m, int n0, i
     }
     const float up = __shfl_down_sync(0xffffffffu, s, 8);
     if (r < 8 && m < M && n0 + r + 8 < N)
-        C[(size_t)m * ldc + (n0 >> 1) + r] = from_f32<OutT>(gate_activate(s, epi) * up);
+        C[(size_t)m * ldc + (n0 >> 1) + r] = from_f32<OutT>(gated_value(s, up, epi));
 }
 
 // grid = (ceil(N/16), S) with clusters of (1, S, 1): blockIdx.y is the CTA's

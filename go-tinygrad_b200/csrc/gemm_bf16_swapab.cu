@@ -304,7 +304,7 @@ swapab_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__
                     OutT* dst = C + (size_t)t * ldc + j;
 #pragma unroll
                     for (int i = 0; i < 4; ++i)
-                        if (j + i < (N >> 1)) dst[i] = from_f32<OutT>(gate_activate(g[i], epi) * u[i]);
+                        if (j + i < (N >> 1)) dst[i] = from_f32<OutT>(gated_value(g[i], u[i], epi));
                 }
             }
         }

@@ -434,8 +434,8 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                     const float g1 = __uint_as_float(v[16 * blk + 2 * q + 1]), u1 = __uint_as_float(v[16 * blk + 9 + 2 * q]);
                                     __nv_bfloat162 h = epi_code == 1 ? __floats2bfloat162_rn(g0 / (1.0f + __expf(-g0)) * u0,
                                                                                              g1 / (1.0f + __expf(-g1)) * u1)
-                                                                     : __floats2bfloat162_rn(gate_activate(g0, epi_code) * u0,
-                                                                                             gate_activate(g1, epi_code) * u1);
+                                                                     : __floats2bfloat162_rn(gated_value(g0, u0, epi_code),
+                                                                                             gated_value(g1, u1, epi_code));
                                     p[q] = *reinterpret_cast<uint32_t*>(&h);
                                 }
                                 const int chunk = 2 * cc + blk;
@@ -476,7 +476,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
 #pragma unroll
                             for (int q = 0; q < 8; ++q) {
                                 const float g = __uint_as_float(v[16 * blk + q]), u = __uint_as_float(v[16 * blk + 8 + q]);
-                                o[8 * blk + q] = __float_as_uint((epi_code == 1 ? g / (1.0f + __expf(-g)) : gate_activate(g, epi_code)) * u);
+                                o[8 * blk + q] = __float_as_uint(epi_code == 1 ? g / (1.0f + __expf(-g)) * u : gated_value(g, u, epi_code));
                             }
                         store_values<OutT, 16>(C + (size_t)row * ldc + (col >> 1), o, min(16, (N - col) / 2), vec_ok);
                     }

@@ -31,6 +31,8 @@ LIBRARIES: Dict[str, str] = {
     "elementwise": "elementwise.cu",
     "gemm_f32": "gemm_f32.cu",
     "attention_simple": "attention_simple.cu",
+    "attention_diff": "attention_diff.cu",
+    "lightning": "lightning.cu",
     "sampling": "sampling.cu",
     "gemm_bf16_mma": "gemm_bf16_mma.cu",
     "gemm_bf16_skinny": "gemm_bf16_skinny.cu",

@@ -8,7 +8,9 @@ is no other route for the same work (no library attention, no CPU path).
 from __future__ import annotations
 
 import ctypes
+import struct
 from ctypes import c_double, c_float, c_int, c_longlong, c_ulonglong, c_void_p
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -30,6 +32,7 @@ _SIGNATURES = {
     "gtg_rope_table": ("elementwise", [_P, _P, _P, _I, _I, _D, _P]),
     "gtg_rope_kv_store": ("elementwise", [_I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _P]),
     "gtg_add_layernorm": ("elementwise", [_I, _P, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
+    "gtg_layernorm_add_layernorm": ("elementwise", [_I, _I, _P, _P, _P, _F, _P, _P, _F, _P, _P, _I, _I, _P]),
     "gtg_activation": ("elementwise", [_I, _P, _I, _I, _I, _I, _P]),
     "gtg_softcap": ("elementwise", [_P, _L, _F, _P]),
     "gtg_hidden_concat": ("elementwise", [_I, _P, _P, _P, _P, _I, _I, _P]),
@@ -70,7 +73,7 @@ _SIGNATURES = {
     "gtg_mlstm_scan": ("mlstm", [_I, _P, _P, _P, _I, _P, _I, _P, _F, _F, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _P]),
     "gtg_rmsnorm_add": ("elementwise", [_I, _I, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
     "gtg_round_rows": ("elementwise", [_I, _P, _P, _L, _P]),
-    "gtg_swiglu_bias": ("elementwise", [_I, _P, _P, _P, _P, _I, _I, _I, _P]),
+    "gtg_swiglu_bias": ("elementwise", [_I, _P, _P, _P, _P, _I, _I, _I, _I, _P]),
     "gtg_add_bias": ("elementwise", [_I, _P, _P, _P, _I, _I, _P]),
     "gtg_sigmoid_gate": ("elementwise", [_I, _P, _I, _P, _I, _I, _I, _I, _P]),
     "gtg_gemm_simt_batched": ("gemm_f32", [_I, _P, _I, _L, _P, _I, _L, _P, _I, _L, _I, _I, _I, _I, _P]),
@@ -88,19 +91,27 @@ _SIGNATURES = {
     "gtg_latent_attention_splits": ("latent", [_I, _I, _I, _I, _I, _I]),
     "gtg_moe_gather": ("experts", [_P, _I, _P, _I, _P, _I, _I, _P]),
     "gtg_gemm_bf16_tcgen05_grouped": ("gemm_bf16_tcgen05", [_P, _I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _I, _P]),
-    "gtg_moe_route": ("experts", [_I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P]),
+    "gtg_moe_route": ("experts", [_I, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _F, _P]),
     "gtg_moe_gather_scaled": ("experts", [_I, _P, _I, _P, _I, _P, _P, _I, _I, _P]),
     "gtg_attention_masked_supports": ("attention_masked", [_I, _I]),
     "gtg_attention_masked_scratch_floats": ("attention_masked", [_I, _I, _I, _I]),
     "gtg_attention_masked_splits": ("attention_masked", [_I, _I, _I, _I, _I, _I, _I]),
     "gtg_attention_masked_bf16": ("attention_masked", [_P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I,
                                                        _F, _I, _I, _P, _I, _P, _F, _I, _P, _P]),
+    "gtg_attention_diff_simple": ("attention_diff", [_I, _P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _F, _I,
+                                                     _F, _F, _F, _P]),
+    "gtg_attention_diff_supports": ("attention_diff", [_I, _I]),
+    "gtg_attention_diff_scratch_floats": ("attention_diff", [_I, _I, _I, _I]),
+    "gtg_attention_diff_splits": ("attention_diff", [_I, _I, _I, _I, _I, _I]),
+    "gtg_attention_diff_bf16": ("attention_diff", [_P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
+                                                   _F, _F, _F, _I, _P, _P]),
+    "gtg_lightning_scan": ("lightning", [_I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
     "gtg_hyper_norm": ("hyper", [_I, _I, _P, _P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P]),
     "gtg_qkv_finish": ("attention_prep", [_I, _P, _I, _P, _P, _I, _I, _F, _P, _P, _F, _P, _I, _P, _P, _P, _L, _P, _I, _P, _P, _P,
-                                          _I, _I, _I, _I, _I, _P]),
+                                          _I, _I, _I, _I, _I, _I, _P]),
     "gtg_moe_arrange": ("experts", [_P, _I, _I, _I, _I, _P, _P, _P, _P]),
     "gtg_moe_product_simt": ("experts", [_I, _I, _P, _I, _P, _I, _P, _I, _L, _P, _I, _P, _I, _I, _I, _P]),
-    "gtg_moe_combine": ("experts", [_I, _P, _I, _P, _P, _P, _I, _I, _I, _P]),
+    "gtg_moe_combine": ("experts", [_I, _P, _I, _P, _P, _P, _I, _I, _I, _P, _I, _I, _P, _P]),
     "gtg_attention_bf16_supports": ("attention_bf16", [_I]),
     "gtg_attention_decode_scratch_floats": ("attention_bf16", [_I, _I, _I, _I]),
     "gtg_attention_decode_plan": ("attention_bf16", [_I, _I, _I, _I, _I, _L, _I, _P, _P]),
@@ -119,6 +130,7 @@ _SIGNATURES = {
 }
 _RESTYPES = {"gtg_attention_decode_scratch_floats": c_longlong,
              "gtg_attention_masked_scratch_floats": c_longlong,
+             "gtg_attention_diff_scratch_floats": c_longlong,
              "gtg_gemm_bf16_swapab_scratch_floats": c_longlong}
 
 _FUNCS = {}
@@ -339,15 +351,17 @@ def normed_pair(a: torch.Tensor, b: torch.Tensor, weight_a: torch.Tensor, weight
                                   _ptr(out), N, H, _stream()), "normed_pair")
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[m,i] = act(gate_up[m,i]) * gate_up[m,I+i], act = silu or another of `ACTIVATIONS`."""
-    _need(activation in ACTIVATIONS, f"swiglu: activation {activation!r} is not known; known: {sorted(ACTIVATIONS)}")
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation="silu") -> None:
+    """out[m,i] = act(gate_up[m,i]) * gate_up[m,I+i], act = silu or another of `ACTIVATIONS`; a
+    `ClampedGate` in its place: that product of the two."""
+    _need(isinstance(activation, ClampedGate) or activation in ACTIVATIONS, f"swiglu: activation {activation!r} is not known; known: {sorted(ACTIVATIONS)}")
     M, two_i = gate_up.shape
     _rows2d(out, "swiglu: out")
     _need(two_i % 2 == 0 and gate_up.is_contiguous()
           and tuple(out.shape) == (M, two_i // 2) and out.dtype == gate_up.dtype,
           "swiglu: gate_up [M, 2I] must be contiguous and out [M, I] of its dtype")
-    _check(_fn("gtg_swiglu")(_dt(out), _ptr(gate_up), _ptr(out), out.stride(0), M, two_i // 2, ACTIVATIONS[activation], _stream()), "swiglu")
+    _check(_fn("gtg_swiglu")(_dt(out), _ptr(gate_up), _ptr(out), out.stride(0), M, two_i // 2,
+                             activation.code if isinstance(activation, ClampedGate) else ACTIVATIONS[activation], _stream()), "swiglu")
 
 
 def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor, amplitude: float = 1.0) -> None:
@@ -434,11 +448,63 @@ def add_layernorm(residual: torch.Tensor, pending: Optional[torch.Tensor], weigh
                                     _ptr(out), _ptr(rows), R, H, _stream()), "add_layernorm")
 
 
+def layernorm_add_layernorm(residual: torch.Tensor, update: torch.Tensor, update_weight: torch.Tensor, update_eps: float,
+                            weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out: torch.Tensor,
+                            rows: Optional[torch.Tensor] = None) -> None:
+    """residual += LN(update) * update_weight; out = LN(residual) * weight (+ bias), LN(x) = (x - mean) /
+    sqrt(var + eps), all in float.  `update` is float32 or of out's dtype.  With `rows` only those rows are
+    read (nothing is written back) and out has len(rows) rows."""
+    H = residual.shape[1]
+    R = rows.numel() if rows is not None else residual.shape[0]
+    _need(residual.dtype == torch.float32 and residual.is_contiguous(), "layernorm_add_layernorm: residual must be contiguous float32")
+    _need(update.is_contiguous() and update.shape == residual.shape and update.dtype in (torch.float32, out.dtype),
+          "layernorm_add_layernorm: update must be contiguous [N, H], float32 or of out's dtype")
+    for name, t in (("update_weight", update_weight), ("weight", weight), ("bias", bias)):
+        _need((t is None and name == "bias") or (t is not None and t.dtype == torch.float32 and t.is_contiguous() and t.numel() == H),
+              f"layernorm_add_layernorm: {name} must be float32 [H]")
+    _need(out.is_contiguous() and tuple(out.shape) == (R, H), "layernorm_add_layernorm: out must be contiguous [rows, H]")
+    if rows is not None:
+        _need(rows.dtype == torch.int32 and rows.is_contiguous(), "layernorm_add_layernorm: rows must be contiguous int32")
+    _check(_fn("gtg_layernorm_add_layernorm")(_dt(out), 1 if update.dtype == torch.float32 else 0, _ptr(residual), _ptr(update),
+                                              _ptr(update_weight), float(update_eps), _ptr(weight), _ptr(bias), float(eps), _ptr(out),
+                                              _ptr(rows), R, H, _stream()), "layernorm_add_layernorm")
+
+
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
 # gate activations whose product act(gate) * up the products' epilogues form, and the epilogue's name
 GATED_EPILOGUES = {"silu": "swiglu", "gelu_tanh": "gated_gelu_tanh", "relu2": "gated_relu2"}
 EPILOGUE_GATED = 32           # a product's epilogue code from here on: the gated product with activation (code - 32) on the gate
 EPILOGUE_ACTIVATION = 16      # a product's epilogue code from here on: the plain product, then activation (code - 16)
+
+
+@dataclass(frozen=True)
+class ClampedGate:
+    """An epilogue of the gated products: g = min(gate, limit), u = up between -limit and limit,
+    g sigmoid(1.702 g) (u + 1).  Its code is the limit's bit pattern."""
+    limit: float
+
+    @property
+    def code(self) -> int:
+        _need(self.limit >= 1.2e-38, f"a clamped gate needs a positive limit, not {self.limit}")
+        return struct.unpack("<i", struct.pack("<f", self.limit))[0]
+
+
+def _is_gated(epilogue) -> bool:
+    return isinstance(epilogue, ClampedGate) or epilogue in GATED_EPILOGUES.values()
+
+
+def _epilogue_code(epilogue) -> int:
+    """What the products' kernels are told for an epilogue's name (or a `ClampedGate`)."""
+    if isinstance(epilogue, ClampedGate):
+        return epilogue.code
+    if epilogue == "swiglu":
+        return 1
+    if epilogue in GATED_EPILOGUES.values():
+        return EPILOGUE_GATED + ACTIVATIONS[epilogue[len("gated_"):]]
+    if epilogue in ACTIVATIONS:
+        return EPILOGUE_ACTIVATION + ACTIVATIONS[epilogue]
+    _need(epilogue == "none", f"unknown epilogue {epilogue!r}")
+    return 0
 
 
 def activation(x: torch.Tensor, kind: str) -> None:
@@ -545,16 +611,21 @@ def hyper_norm(copies: torch.Tensor, weight: torch.Tensor, eps: float, out: torc
 def qkv_finish(sums: torch.Tensor, bias: Optional[torch.Tensor], cos_sin: Optional[torch.Tensor], n_heads: int, kv,
                q_out: torch.Tensor, token_seq, slots, positions, *, unit_norm: bool = False, eps: float = 0.0,
                v_first: Optional[torch.Tensor] = None, v_keep: Optional[torch.Tensor] = None, blend: float = 0.0,
-               gate_out: Optional[torch.Tensor] = None, store: bool = True) -> None:
+               gate_out: Optional[torch.Tensor] = None, store: bool = True, maps: int = 1,
+               queries_only: bool = False) -> None:
     """From the float sums of a fused projection [N, q | k | v | gate]: biases added, the first
     channels of query and key heads rotated (half-split pairs, as many as the table has),
     optionally each head divided by its root mean square, values blended with `v_first`
     ((1 - blend) v + blend v_first; float32 [N, n_kv * value_dim]) or kept in `v_keep`
     unblended, gate columns turned into sigmoid factors (`gate_out` float32 [N, n_heads]);
-    queries to `q_out`, keys and values into the cache `kv` (its head_dim and value_dim)."""
+    queries to `q_out`, keys and values into the cache `kv` (its head_dim and value_dim).  `maps`: a query
+    or key head is that many equal parts side by side, each rotated on its own first channels.
+    `queries_only`: the sums have no key and value columns (a layer that reads another's cache)."""
     _rows2d(sums, "qkv_finish: sums"); _rows2d(q_out, "qkv_finish: q_out")
     N = sums.shape[0]
-    hd, vd, n_kv = kv.head_dim, kv.value_dim, kv.n_kv_heads
+    hd, vd, n_kv = kv.head_dim, kv.value_dim, 0 if queries_only else kv.n_kv_heads
+    store = store and not queries_only
+    _need(maps >= 1 and hd % maps == 0, "qkv_finish: a head must be a whole number of maps")
     biased = n_heads * hd + n_kv * (hd + vd)
     width = biased + (n_heads if gate_out is not None else 0)
     _need(sums.dtype == torch.float32 and sums.shape[1] >= width, f"qkv_finish: sums must be float32 with {width} columns at least")
@@ -564,7 +635,7 @@ def qkv_finish(sums: torch.Tensor, bias: Optional[torch.Tensor], cos_sin: Option
         _need(cos_sin.dtype == torch.float32 and cos_sin.is_contiguous() and cos_sin.shape[0] == N and cos_sin.shape[2] == 2,
               "qkv_finish: the rotation table must be float32 [N, pairs, 2]")
         rot = 2 * cos_sin.shape[1]
-        _need(rot <= hd, "qkv_finish: more rotated channels than a head has")
+        _need(rot <= hd // maps, "qkv_finish: more rotated channels than a head has")
     _need(q_out.dtype == kv.k.dtype and q_out.shape[0] == N and q_out.shape[1] >= n_heads * hd, "qkv_finish: q_out must be [N, n_heads * head_dim] of the cache's dtype")
     for t, name in ((v_first, "v_first"), (v_keep, "v_keep")):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and tuple(t.shape) == (N, n_kv * vd)), f"qkv_finish: {name} must be float32 [N, n_kv * value_dim]")
@@ -576,7 +647,7 @@ def qkv_finish(sums: torch.Tensor, bias: Optional[torch.Tensor], cos_sin: Option
     _check(_fn("gtg_qkv_finish")(_dt(q_out), _ptr(sums), sums.stride(0), _ptr(bias), _ptr(cos_sin), rot, 1 if unit_norm else 0, float(eps),
                                  _ptr(v_first), _ptr(v_keep), float(blend), _ptr(q_out), q_out.stride(0), _ptr(gate_out),
                                  _ptr(kv.k) if store else None, _ptr(kv.v) if store else None, kv.page_stride, _ptr(kv.block_table),
-                                 kv.table_stride, _ptr(token_seq), _ptr(slots), _ptr(positions), N, n_heads, n_kv, hd, vd, _stream()),
+                                 kv.table_stride, _ptr(token_seq), _ptr(slots), _ptr(positions), N, n_heads, n_kv, hd, vd, int(maps), _stream()),
            "qkv_finish")
 
 
@@ -588,9 +659,10 @@ def round_rows(x: torch.Tensor, out: torch.Tensor) -> None:
 
 
 def swiglu_bias(gate_up: torch.Tensor, gate_bias: Optional[torch.Tensor], up_bias: Optional[torch.Tensor],
-                out: torch.Tensor) -> None:
+                out: torch.Tensor, epilogue="swiglu") -> None:
     """out[m,i] = silu(gate_up[m,i] + gate_bias[i]) * (gate_up[m,I+i] + up_bias[i]) from a
-    product's float32 sums [M, 2I]."""
+    product's float32 sums [M, 2I]; another gated `epilogue`: that product of the two."""
+    _need(_is_gated(epilogue), f"swiglu_bias: {epilogue!r} is not a gated epilogue")
     _rows2d(out, "swiglu_bias: out")
     M, two_i = gate_up.shape
     I = two_i // 2
@@ -599,7 +671,7 @@ def swiglu_bias(gate_up: torch.Tensor, gate_bias: Optional[torch.Tensor], up_bia
     for name, t in (("gate_bias", gate_bias), ("up_bias", up_bias)):
         _need(t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == I), f"swiglu_bias: {name} must be float32 [I]")
     _check(_fn("gtg_swiglu_bias")(_dt(out), _ptr(gate_up), _ptr(gate_bias), _ptr(up_bias), _ptr(out), out.stride(0), M, I,
-                                  _stream()), "swiglu_bias")
+                                  _epilogue_code(epilogue), _stream()), "swiglu_bias")
 
 
 def add_bias(x: torch.Tensor, bias: torch.Tensor, out: torch.Tensor) -> None:
@@ -834,6 +906,34 @@ def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.T
                                  _ptr(slots), int(n_seqs), heads, d, dv, 1 if one_token_each else 0, _stream()), "mlstm_scan")
 
 
+LIGHTNING_MAX_KEY_DIM = 512   # most key channels a head of linear attention may have (16 rows a lane, 32 lanes)
+
+
+def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                   cu_seqlens, slots, n_seqs: int, one_token_each: bool = False) -> None:
+    """Linear attention with a fixed decay per head (csrc/lightning.cu): S <- decay S + k v^T, out = S^T q;
+    q, k [n, heads * d] and v [n, heads * dv], columns of one matrix; decay float32 [heads]; state float32
+    [slots, heads, d, dv], read and left per sequence; out float32 [n, heads * dv].  `one_token_each`: row
+    b is sequence b's only token."""
+    for name, t in (("q", q), ("k", k), ("v", v), ("out", out)):
+        _rows2d(t, f"lightning_scan: {name}")
+    heads = decay.numel()
+    n = q.shape[0]
+    _need(q.shape[1] % heads == 0 and v.shape[1] % heads == 0 and k.shape == q.shape and v.shape[0] == n, "lightning_scan: q, k and v do not fit the heads")
+    d, dv = q.shape[1] // heads, v.shape[1] // heads
+    _need(q.dtype == k.dtype == v.dtype and q.stride(0) == k.stride(0) == v.stride(0), "lightning_scan: q, k and v must be columns of one matrix")
+    _need(decay.dtype == torch.float32 and decay.is_contiguous(), "lightning_scan: decay must be float32 [heads]")
+    _need(out.dtype == torch.float32 and tuple(out.shape) == (n, heads * dv), "lightning_scan: out must be float32 [n, heads * dv]")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, d, dv), "lightning_scan: state must be float32 [slots, heads, d, dv]")
+    _need(d <= LIGHTNING_MAX_KEY_DIM, f"lightning_scan: heads of {d} key channels exceed {LIGHTNING_MAX_KEY_DIM}")
+    _int32("lightning_scan", cu_seqlens, slots)
+    if one_token_each:
+        _need(n == n_seqs, "lightning_scan: one token each means as many rows as sequences")
+    _check(_fn("gtg_lightning_scan")(_dt(q), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), _ptr(state), _ptr(out), out.stride(0),
+                                     _ptr(cu_seqlens), _ptr(slots), int(n_seqs), heads, d, dv, 1 if one_token_each else 0, _stream()),
+           "lightning_scan")
+
+
 # ------------------------------------------------------------- recurrent mixers
 def _int32(name: str, *tensors) -> None:
     for t in tensors:
@@ -954,7 +1054,7 @@ def interleave_gate_up(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str = "auto",
-           epilogue: str = "none") -> None:
+           epilogue="none") -> None:
     """out[M,N] = x[M,K] . w[N,K]^T.  float32 operands take the true 32-bit
     kernel; bfloat16 operands accumulate in float and write bfloat16 or float32.
     `kind` picks the bfloat16 kernel: "auto" (by the number of rows), "skinny"
@@ -963,13 +1063,14 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str = "aut
     or "tiled" (warp-level MMA).  epilogue="swiglu" (bfloat16, not "tiled"): w is laid out by
     `interleave_gate_up` and out[M, N/2] = silu(gate) * up, computed from the
     float accumulators; epilogue="gated_gelu_tanh" | "gated_relu2": the same with that
-    activation on the gate.  epilogue="relu2" | "gelu_tanh" | "silu": out[M, N] is that
+    activation on the gate; a `ClampedGate`: that gated product.  epilogue="relu2" | "gelu_tanh" | "silu": out[M, N] is that
     activation of the product, applied to the float sums inside the tensor-core
     kernels, by the `activation` kernel behind the others."""
     _rows2d(x, "linear: x"); _rows2d(w, "linear: w"); _rows2d(out, "linear: out")
     M, K = x.shape
     N = w.shape[0]
-    if epilogue in ACTIVATIONS:
+    gated = _is_gated(epilogue)
+    if not gated and epilogue in ACTIVATIONS:
         fused = (x.dtype == torch.bfloat16 and kind != "tiled" and K % 8 == 0 and x.stride(0) % 8 == 0
                  and w.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
                  and out.data_ptr() % 16 == 0 and out.stride(0) % (4 if out.dtype == torch.float32 else 8) == 0)
@@ -977,8 +1078,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str = "aut
             linear(x, w, out, kind=kind)
             activation(out, epilogue)
             return
-    gated = epilogue in GATED_EPILOGUES.values()
-    _need(epilogue == "none" or gated or epilogue in ACTIVATIONS, f"linear: unknown epilogue {epilogue!r}")
+    epi_code = _epilogue_code(epilogue)
     n_out = N // 2 if gated else N
     _need(w.shape[1] == K and tuple(out.shape) == (M, n_out),
           f"linear: shapes {tuple(x.shape)} x {tuple(w.shape)} -> {tuple(out.shape)} (epilogue {epilogue})")
@@ -1011,8 +1111,6 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, kind: str = "aut
         most = WARP_LEVEL_MAX_ROWS if kind == "skinny" else SKINNY_MAX_ROWS
         _need(M <= most, f"linear: the weight-streaming kernel {kind!r} takes at most {most} rows")
     out_f32 = 1 if out.dtype == torch.float32 else 0
-    epi_code = (1 if epilogue == "swiglu" else EPILOGUE_GATED + ACTIVATIONS[epilogue[len("gated_"):]] if gated
-                else EPILOGUE_ACTIVATION + ACTIVATIONS[epilogue] if epilogue in ACTIVATIONS else 0)
     if kind == "tiled":
         _need(epilogue == "none", "linear: the warp-level kernel has no fused epilogue")
         code = _fn(symbol)(_ptr(x), x.stride(0), _ptr(w), w.stride(0), _ptr(out), out.stride(0),
@@ -1294,6 +1392,68 @@ def attention_masked_bf16(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: int,
                                             float(scale), int(window), int(chunk), _ptr(gate), int(n_splits), _ptr(scratch),
                                             float(softcap), int(gate_ld), _ptr(slopes), _stream()),
            "attention_masked_bf16")
+
+
+def attention_diff_simple(q: torch.Tensor, out: torch.Tensor, kv, token_seq, slots, positions, n_heads: int, scale: float,
+                          lam: float, out_scale: float, eps: float, window: int = 0) -> None:
+    """Differential attention, one warp per (token, head), either dtype: q [N, heads * 2 d] (a head's map
+    1, then its map 2), key rows of 2 d, value rows of kv.value_dim channels; with a1 and a2 the maps'
+    outputs and o = a1 - lam a2, out = o / sqrt(mean(o^2) + eps) * out_scale per head."""
+    _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
+    N, d, vd = q.shape[0], kv.head_dim // 2, kv.value_dim
+    _need(kv.head_dim % 2 == 0, "attention_diff: key rows must hold two maps")
+    _need(kv.k.dtype == q.dtype == out.dtype, "attention: q, out and the cache must share a dtype")
+    _need(q.shape[1] >= n_heads * 2 * d and out.shape[1] >= n_heads * vd, "attention: q or out is too narrow")
+    _int32("attention_diff", token_seq, slots, positions)
+    _check_access("attention_diff_simple", 0, kv, slots, positions, token_seq, n_items=N)
+    _check(_fn("gtg_attention_diff_simple")(_dt(q), _ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kv.k), _ptr(kv.v),
+                                            kv.page_stride, _ptr(kv.block_table), kv.table_stride, _ptr(token_seq), _ptr(slots),
+                                            _ptr(positions), N, n_heads, kv.n_kv_heads, d, vd, float(scale), int(window),
+                                            float(lam), float(out_scale), float(eps), _stream()), "attention_diff_simple")
+
+
+def attention_diff_supports(kv) -> bool:
+    """Whether `attention_diff_bf16` takes this cache entry."""
+    return (kv.k.dtype == torch.bfloat16 and kv.head_dim % 2 == 0 and kv.page_stride % 8 == 0
+            and bool(_fn("gtg_attention_diff_supports")(kv.head_dim // 2, kv.value_dim)))
+
+
+def attention_diff_bf16(q: torch.Tensor, out: torch.Tensor, kv, cu_seqlens, slots, start_pos, n_seqs: int, max_q_len: int,
+                        n_heads: int, scale: float, lam: float, out_scale: float, eps: float, window: int = 0,
+                        n_splits: int = 1, scratch: Optional[torch.Tensor] = None) -> None:
+    """The tensor-core form of `attention_diff_simple`; `n_splits` > 1 cuts every tile's pages into that
+    many shares, merged through `scratch` (float32, `gtg_attention_diff_scratch_floats`)."""
+    _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
+    N, d, vd = q.shape[0], kv.head_dim // 2, kv.value_dim
+    _need(q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and attention_diff_supports(kv), "attention_diff_bf16: cache entry not supported")
+    _need(q.shape[1] >= n_heads * 2 * d and out.shape[1] >= n_heads * vd, "attention: q or out is too narrow")
+    _int32("attention_diff", cu_seqlens, slots, start_pos)
+    if n_splits > 1:
+        need = int(_fn("gtg_attention_diff_scratch_floats")(N, n_heads, vd, n_splits))
+        _need(scratch is not None and scratch.dtype == torch.float32 and scratch.is_contiguous() and scratch.numel() >= need,
+              f"attention_diff_bf16: {n_splits} shares need {need} floats of scratch")
+    _check_access("attention_diff_bf16", 2, kv, slots, start_pos=start_pos, cu_seqlens=cu_seqlens, n_items=n_seqs)
+    _check(_fn("gtg_attention_diff_bf16")(_ptr(q), q.stride(0), _ptr(out), out.stride(0), _ptr(kv.k), _ptr(kv.v), kv.page_stride,
+                                          _ptr(kv.block_table), kv.table_stride, _ptr(cu_seqlens), _ptr(slots), _ptr(start_pos),
+                                          int(n_seqs), int(max_q_len), N, n_heads, kv.n_kv_heads, d, vd, float(scale), int(window),
+                                          float(lam), float(out_scale), float(eps), int(n_splits), _ptr(scratch), _stream()),
+           "attention_diff_bf16")
+
+
+def attention_diff(q: torch.Tensor, out: torch.Tensor, kv, ctx, n_heads: int, scale: float, lam: float, out_scale: float,
+                   eps: float, window: int = 0) -> None:
+    """Differential attention of a step (`ctx`: its context) by the kernel that takes its sizes."""
+    if (q.dtype == torch.bfloat16 and attention_diff_supports(kv) and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
+            and out.stride(0) % 2 == 0 and scale > 0):
+        splits = int(_fn("gtg_attention_diff_splits")(ctx.n_seqs, ctx.max_q_len, n_heads, kv.n_kv_heads, ctx.max_kv_len, int(window)))
+        scratch = None
+        if splits > 1:
+            scratch = ctx.rt.empty(int(_fn("gtg_attention_diff_scratch_floats")(q.shape[0], n_heads, kv.value_dim, splits)),
+                                   dtype=torch.float32)
+        attention_diff_bf16(q, out, kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, ctx.n_seqs, ctx.max_q_len, n_heads, scale, lam,
+                            out_scale, eps, window, splits, scratch)
+        return
+    attention_diff_simple(q, out, kv, ctx.token_seq, ctx.slots, ctx.positions, n_heads, scale, lam, out_scale, eps, window)
 
 
 def attention_prefill_bf16(q, out, kv, cu_seqlens, slots, start_pos, n_seqs: int, max_q_len: int,
@@ -1578,14 +1738,17 @@ def expanded_attention_bf16(q: torch.Tensor, runs: torch.Tensor, out: torch.Tens
 MOE_TILE_ROWS = 64
 
 
-MOE_SCORING = {"softmax_chosen": 0, "sigmoid": 1}
+MOE_SCORING = {"softmax_chosen": 0, "sigmoid": 1, "softmax_all": 2}
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor], chosen: torch.Tensor,
-              weights: torch.Tensor, scoring: str = "softmax_chosen") -> None:
+              weights: torch.Tensor, scoring: str = "softmax_chosen", correction: Optional[torch.Tensor] = None,
+              weight_scale: float = 1.0) -> None:
     """Router logits x . router^T + bias in float; chosen[n, :] = the `top` largest
     (ties: the lower index), weights[n, :] = softmax over those logits alone
-    ("softmax_chosen") or each chosen logit's own sigmoid ("sigmoid")."""
+    ("softmax_chosen") or each chosen logit's own sigmoid ("sigmoid").  "softmax_all": s = softmax over
+    all logits, the largest s + correction (float32 [E]) are chosen, and the weights are the chosen s
+    over their sum (+ 1e-20), times `weight_scale`."""
     _need(scoring in MOE_SCORING, f"moe_route: scoring {scoring!r} is not known; known: {sorted(MOE_SCORING)}")
     _rows2d(x, "moe_route: x")
     N, H = x.shape
@@ -1595,8 +1758,11 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, bias: Optional[torch.Tensor
     _need(chosen.dtype == torch.int32 and chosen.is_contiguous() and weights.dtype == torch.float32 and weights.is_contiguous()
           and tuple(chosen.shape) == (N, top) and tuple(weights.shape) == (N, top) and 0 < top <= E,
           "moe_route: chosen int32 [N, top] and weights float32 [N, top]")
+    _need((correction is None and weight_scale == 1.0) or scoring == "softmax_all", "moe_route: a correction and a scale go with scores over all outputs")
+    _need(correction is None or (correction.dtype == torch.float32 and correction.is_contiguous() and correction.numel() == E),
+          "moe_route: correction must be float32 [E]")
     _check(_fn("gtg_moe_route")(_dt(x), _ptr(x), x.stride(0), _ptr(router), _ptr(bias), _ptr(chosen), _ptr(weights), N, H, E, top,
-                                MOE_SCORING[scoring], _stream()), "moe_route")
+                                MOE_SCORING[scoring], _ptr(correction), float(weight_scale), _stream()), "moe_route")
 
 
 def moe_tiles_cap(n_items: int, n_experts: int, tile: int = MOE_TILE_ROWS) -> int:
@@ -1607,7 +1773,8 @@ def moe_tiles_cap(n_items: int, n_experts: int, tile: int = MOE_TILE_ROWS) -> in
 def moe_arrange(chosen: torch.Tensor, n_experts: int, row_item: torch.Tensor, item_row: torch.Tensor,
                 tile_expert: torch.Tensor, tile: int = MOE_TILE_ROWS) -> None:
     """Order the (token, expert) pairs by expert, every expert's rows padded to whole
-    tiles: row_item[row] = pair or -1, item_row[pair] = row, tile_expert[tile] = expert or -1."""
+    tiles: row_item[row] = pair or -1, item_row[pair] = row, tile_expert[tile] = expert or -1.
+    A choice of n_experts or more stands for no expert: its pair has no row, item_row[pair] = -1."""
     n_items = chosen.numel()
     cap = tile_expert.numel()
     _int32("moe_arrange", chosen, row_item, item_row, tile_expert)
@@ -1647,35 +1814,35 @@ def moe_product_fused_supports(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def moe_product(a: torch.Tensor, row_item: torch.Tensor, item_div: int, w: torch.Tensor, tile_expert: torch.Tensor,
-                out: torch.Tensor, epilogue: str = "none") -> None:
+                out: torch.Tensor, epilogue="none") -> None:
     """out[row, :] = a[source(row), :] . w[expert of the row's tile]^T over arranged
     rows.  item_div > 0: the source is the pair's token, row_item[row] // item_div
     (a holds tokens); 0: the row itself (a holds arranged rows, zeros in its padding
     rows: `moe_gather`), which in tiles of 128 takes the prompt-sized tensor-memory
     product.  w [E, N, K].  The tile is out's rows over tile_expert's length: 64, or 128 on the tensor
     cores.  epilogue="swiglu" (tensor cores only: `moe_product_fused_supports`):
-    every w[e] is laid out by `interleave_gate_up` and out [rows, N/2] = silu(gate) * up.
-    epilogue="relu2" | "gelu_tanh" | "silu": that activation of the product, applied to the float
+    every w[e] is laid out by `interleave_gate_up` and out [rows, N/2] = silu(gate) * up;
+    a `ClampedGate`: that gated product.  epilogue="relu2" | "gelu_tanh" | "silu": that activation of the product, applied to the float
     sums inside the tensor-core kernels, by the `activation` kernel behind the plain one."""
     _rows2d(a, "moe_product: a"); _rows2d(out, "moe_product: out")
     E, N, K = w.shape
     cap = tile_expert.numel()
     tile = out.shape[0] // max(cap, 1)
-    _need(epilogue in ("none", "swiglu") or epilogue in ACTIVATIONS, f"moe_product: unknown epilogue {epilogue!r}")
-    if epilogue in ACTIVATIONS and not moe_product_fused_supports(a, w):
+    gated = _is_gated(epilogue)
+    epi_code = _epilogue_code(epilogue)
+    if not gated and epilogue in ACTIVATIONS and not moe_product_fused_supports(a, w):
         # the plain product has no epilogue: the activation runs behind it
         moe_product(a, row_item, item_div, w, tile_expert, out)
         activation(out, epilogue)
         return
-    n_out = N // 2 if epilogue == "swiglu" else N
-    epi_code = 1 if epilogue == "swiglu" else EPILOGUE_ACTIVATION + ACTIVATIONS[epilogue] if epilogue in ACTIVATIONS else 0
+    n_out = N // 2 if gated else N
     _need(w.is_contiguous() and a.dtype == w.dtype and a.shape[1] == K, "moe_product: a [*, K] and contiguous w [E, N, K] of one dtype")
     _need(tuple(out.shape) == (cap * tile, n_out) and out.dtype in (a.dtype, torch.float32), "moe_product: out must be [tiles * tile, N]")
     _need(item_div > 0 or a.shape[0] == out.shape[0], "moe_product: a must hold the arranged rows")
     _int32("moe_product", row_item, tile_expert)
     if moe_product_fused_supports(a, w):
         _need(tile in (64, 128), f"moe_product: tiles of 64 or 128 rows, not {tile}")
-        _need(epilogue != "swiglu" or N % 16 == 0, "moe_product: the fused gated silu needs a multiple of 16 rows per expert")
+        _need(not gated or N % 16 == 0, "moe_product: a fused gated product needs a multiple of 16 rows per expert")
         if (tile == 128 and item_div == 0 and out.data_ptr() % 16 == 0
                 and out.stride(0) % (4 if out.dtype == torch.float32 else 8) == 0):
             # arranged rows in tiles of 128: the prompt-sized product (tensor copies, tensor memory)
@@ -1695,9 +1862,11 @@ def moe_product(a: torch.Tensor, row_item: torch.Tensor, item_div: int, w: torch
                                        _stream()), "moe_product")
 
 
-def moe_combine(y: torch.Tensor, item_row: torch.Tensor, weights: Optional[torch.Tensor], out: torch.Tensor) -> None:
+def moe_combine(y: torch.Tensor, item_row: torch.Tensor, weights: Optional[torch.Tensor], out: torch.Tensor,
+                x: Optional[torch.Tensor] = None, base: Optional[torch.Tensor] = None) -> None:
     """out[t, :] = sum_k weights[t, k] * y[item_row[t * top + k], :] (float sums, k in
-    order; out float32 or bfloat16).  weights None: the plain sum of a token's rows."""
+    order; out float32 or bfloat16).  weights None: the plain sum of a token's rows.  A pair without a
+    row (item_row -1) stands for the token's own input x[t, :].  `base`: float32 [N, H], added last."""
     _rows2d(y, "moe_combine: y")
     N = out.shape[0]
     top = item_row.numel() // max(N, 1)
@@ -1706,7 +1875,13 @@ def moe_combine(y: torch.Tensor, item_row: torch.Tensor, weights: Optional[torch
           and (weights is None or (weights.dtype == torch.float32 and weights.is_contiguous() and tuple(weights.shape) == (N, top))),
           "moe_combine: y float32 [rows, H], weights float32 [N, top], out [N, H]")
     _int32("moe_combine", item_row)
-    _check(_fn("gtg_moe_combine")(_dt(out), _ptr(y), y.stride(0), _ptr(item_row), _ptr(weights), _ptr(out), N, H, top, _stream()),
+    if x is not None:
+        _rows2d(x, "moe_combine: x")
+        _need(tuple(x.shape) == (N, H) and (out.dtype == torch.float32 or x.dtype == out.dtype), "moe_combine: x must be [N, H] of out's dtype (any beside a float32 out)")
+    _need(base is None or (base.dtype == torch.float32 and base.is_contiguous() and tuple(base.shape) == (N, H)), "moe_combine: base must be contiguous float32 [N, H]")
+    _check(_fn("gtg_moe_combine")(_dt(out), _ptr(y), y.stride(0), _ptr(item_row), _ptr(weights), _ptr(out), N, H, top, _ptr(x),
+                                  x.stride(0) if x is not None else 0,
+                                  _dt(x) if x is not None else _dt(out), _ptr(base), _stream()),
            "moe_combine")
 
 

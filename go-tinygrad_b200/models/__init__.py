@@ -1,2 +1,2 @@
 """Architectures the library ships with.  Importing this package registers them."""
-from . import llama, megerax, mererax, ropovik, senupel, zotolix  # noqa: F401  (registration)
+from . import letanex, llama, megerax, mererax, ropovik, senupel, zotolix  # noqa: F401  (registration)

@@ -64,6 +64,15 @@ times 1 + coef ln(floor((p + 1) / every) + 1) at position p; and ``distance_slop
 True takes 2^(-8 (h + 1) / n_heads) times the distance between query and key off the
 scores of head h.  A mixer of this family can be handed its projected rows by a part
 that projects for several (`input_matrix`, `forward_projected`).
+
+A fourth option, differential attention (``differential``: {"diff": number, "lq1" | "lk1" |
+"lq2" | "lk2": tensor names of [head_dim] vectors}; `_forward_differential`): every query and
+key head has two parts of ``head_dim`` channels side by side, each pair of parts is a softmax
+attention of its own over the head's values, and with a1 and a2 their outputs and lambda =
+exp(sum(lq1 lk1)) - exp(sum(lq2 lk2)) + diff a head's output is o = a1 - lambda a2 divided by
+its root mean square over the head (eps ``norm_eps``) and times 1 - diff.  A rotation turns the
+first channels of every part.  It goes with ``value_dim`` and ``window``; with ``own_kv`` False the
+layer reads another run's cache with queries and a lambda of its own.
 """
 from __future__ import annotations
 
@@ -146,7 +155,15 @@ class GQAttention(Mixer):
                                 or not self.own_kv or self.value_dim != self.head_dim or self.position.kind != "none"):
             raise ValueError("norms over whole rows of queries and keys are built for unrotated keys that are the values too, without "
                              "the other options")
-        self.general = not self.rows_route and bool(self.value_dim != self.head_dim or self.bias_names or self.qk_norm or self.chunk
+        differential = self.p.get("differential")
+        self.differential = dict(differential) if differential else None
+        self.maps = 2 if self.differential else 1         # parts of a query or key head
+        if self.differential and (self.conv_route or self.bias_names or self.qk_norm or self.chunk or self.gate_name or self.blend
+                                  or self.v_from_k or self.temperature or self.sloped):
+            raise ValueError("differential attention is built with a rotation, values of their own width and a window only")
+        self.lam = 0.0
+        self.q_dim, self.kv_dim = self.q_dim * self.maps, self.kv_dim * self.maps
+        self.general = not self.rows_route and not self.differential and bool(self.value_dim != self.head_dim or self.bias_names or self.qk_norm or self.chunk
                             or self.gate_name or self.blend or self.conv_route)
         if self.conv_route and (self.qk_norm == "unit" or self.chunk or self.gate_name or self.blend or self.v_from_k):
             raise ValueError("convolved projections, weighted head norms, capped scores and the gate on all channels are "
@@ -171,6 +188,8 @@ class GQAttention(Mixer):
             if not self.v_from_k:
                 specs.append(WeightSpec(self.names["v"], (self.v_width, self.hidden)))
         specs.append(WeightSpec(self.names["o"], (self.hidden, self.n_heads * self.value_dim)))
+        if self.differential:
+            specs += [WeightSpec(str(self.differential[k]), (self.head_dim,), role="parameter", std=0.1) for k in ("lq1", "lk1", "lq2", "lk2")]
         if self.bias_names:
             specs += [WeightSpec(name, (size,), role="parameter", std=0.02)
                       for name, size in zip(self.bias_names, (self.q_dim, self.kv_dim, self.v_width))]
@@ -209,6 +228,8 @@ class GQAttention(Mixer):
             return requests
         if not self.own_kv:
             return []
+        if self.differential:
+            return [KVRequest(self.n_kv, 2 * self.head_dim, self.cache_window, value_dim=self.value_dim)]
         if self.general:
             return [KVRequest(self.n_kv, self.head_dim, self.cache_window, value_dim=self.value_dim, chunk=self.chunk)]
         return [KVRequest(self.n_kv, self.head_dim, self.cache_window)]
@@ -224,7 +245,7 @@ class GQAttention(Mixer):
         if self.out_gate_name:
             parts.append(tensors[self.out_gate_name])
         rows = sum(p.shape[0] for p in parts)
-        if (self.general or self.rows_route) and rows % 8:
+        if (self.general or self.rows_route or self.differential) and rows % 8:
             # whole groups of 8 rows, so that the products' float sums keep rows of a multiple of 32 bytes
             parts.append(torch.zeros((8 - rows % 8, self.hidden), dtype=parts[0].dtype, device=parts[0].device))
         if not self.shares_input:
@@ -234,6 +255,9 @@ class GQAttention(Mixer):
         self.w_o = rt.matrix(tensors[self.names["o"]])
         if self.bias_names:
             self.bias = rt.vector(torch.cat([tensors[name].reshape(-1).to(torch.float32) for name in self.bias_names]))
+        if self.differential:
+            lq1, lk1, lq2, lk2 = (tensors[str(self.differential[k])].to(torch.float64) for k in ("lq1", "lk1", "lq2", "lk2"))
+            self.lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + float(self.differential["diff"])
         if self.blend and self.blend["role"] == "blend":
             self.blend_weight = float(tensors[str(self.blend["weight"])].to(torch.float32))
         if self.conv:
@@ -329,11 +353,31 @@ class GQAttention(Mixer):
             return out
         return emit_update(mixed, self.w_o, ctx)
 
+    def _forward_differential(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        rt, kv, n = ctx.rt, cache.kv, x.shape[0]
+        sums = rt.empty(n, self.w_qkv.shape[0], dtype=torch.float32)
+        ops.linear(x, self.w_qkv, sums)
+        rotation = self.position.rotation(ctx)
+        if rotation is not None and self.position.pairing != "half":
+            raise ValueError("differential attention rotates half-split pairs only")
+        q = rt.empty(n, (self.q_dim + 7) // 8 * 8)[:, : self.q_dim]
+        ops.qkv_finish(sums, None, rotation, self.n_heads, kv, q, ctx.token_seq, ctx.slots, ctx.positions,
+                       store=cache.writes, maps=2, queries_only=not self.own_kv)
+        ctx.trace("q_attn", q)
+        width = self.n_heads * self.value_dim
+        mixed = rt.empty(n, (width + 7) // 8 * 8)[:, : width]
+        ops.attention_diff(q, mixed, kv, ctx, self.n_heads, self.scale, self.lam, 1.0 - float(self.differential["diff"]),
+                           self.norm_eps, window=self.window or 0)
+        ctx.trace("attn", mixed)
+        return emit_update(mixed, self.w_o, ctx)
+
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
         rt = ctx.rt
         kv = cache.kv
-        if kv is None or kv.n_kv_heads != self.n_kv or kv.head_dim != self.head_dim or kv.value_dim != self.value_dim:
+        if kv is None or kv.n_kv_heads != self.n_kv or kv.head_dim != self.maps * self.head_dim or kv.value_dim != self.value_dim:
             raise ValueError("attention was given a cache entry that does not match its heads")
+        if self.differential:
+            return self._forward_differential(x, ctx, cache)
         if self.rows_route:
             return self._forward_rows(x, ctx, cache)
         if self.conv_route:

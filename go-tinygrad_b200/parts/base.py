@@ -289,7 +289,11 @@ class ResidualStream:
     with a weight of its own while the copies are remixed: `pending_links` holds
     (mix [S, S] indexed [from, to], out [S]) for it, x_t <- sum_s mix[s, t] x_s +
     out[t] pending.  A norm that is handed such a stream applies the update and
-    norms the copies' sum (`ops.hyper_norm`)."""
+    norms the copies' sum (`ops.hyper_norm`).
+
+    `pending_norm`, where set, is a layer norm (weight, eps) that the pending update passes before
+    it is added: a block whose sublayers stand between two norms leaves it to the next norm, which
+    does both in one pass (`ops.layernorm_add_layernorm`).  The pending update may then be float32."""
 
     def __init__(self, residual: torch.Tensor, pending: Optional[torch.Tensor] = None):
         self.residual = residual
@@ -297,6 +301,7 @@ class ResidualStream:
         self.image: Optional[torch.Tensor] = None
         self.copies: Optional[torch.Tensor] = None
         self.pending_links = None
+        self.pending_norm: Optional[Tuple[torch.Tensor, float]] = None
 
 
 class JointUpdate:
@@ -350,7 +355,8 @@ def emit_update(x: torch.Tensor, w: Optional[torch.Tensor], ctx: "StepContext") 
     is added there and None is returned in its place: it never goes through
     memory, and the norm that follows has nothing left to add.  Within a joint
     update (`ctx.joint`) the operand already lies where the block wants it: nothing
-    happens here and None is returned."""
+    happens here and None is returned.  Where the block takes float updates
+    (`ctx.float_updates`) the product's sums are returned as they are."""
     if ctx.joint is not None:
         return None
     stream = ctx.update_into
@@ -358,7 +364,7 @@ def emit_update(x: torch.Tensor, w: Optional[torch.Tensor], ctx: "StepContext") 
             and ops.linear_add_residual(x, w, stream.residual)):
         stream.image = None
         return None
-    out = ctx.rt.empty(x.shape[0], w.shape[0])
+    out = ctx.rt.empty(x.shape[0], w.shape[0], dtype=torch.float32 if ctx.float_updates else None)
     ops.linear(x, w, out)
     return out
 

@@ -29,6 +29,15 @@ next sublayer (`ResidualStream.image`); a part may leave the bias of its last
 projection for that kernel to add (`StepContext.update_bias`).  Nothing is left pending.  The reference
 has no such arrangement.
 
+``sandwich_norm``: x += norm1b(mixer(norm1(x))); x += norm2b(feed_forward(norm2(x))): every
+sublayer stands between two norms.  The four nested specs of ``pre_norm`` and
+``mixer_output_norm`` and ``feed_forward_output_norm``, of kind ``layernorm`` without a
+bias; the feed-forward and its two norms may be None.  As in ``pre_norm`` the
+additions are not done here: an update is left pending together with the norm it has
+to pass (`ResidualStream.pending_norm`), in float32 where the part can leave it so, and the
+next norm does both norms and the addition in one pass.  The reference has no such
+arrangement.
+
 ``hyper_connections``: the hidden state in S copies x_1..x_S (all equal to the
 embedding output at the start).  Sublayer q (the mixer, then the feed-forward)
 reads u = sum_s in_q[s] x_s through its norm, and its output y goes back as
@@ -65,11 +74,21 @@ from ..weights.binder import WeightSpec
 from .base import Block, JointUpdate, ResidualStream, Runtime, StepContext, emit_update, register_part
 
 
+def _pending(stream: ResidualStream):
+    """What is pending on the stream, in float32 and through the norm it has to pass, as a value."""
+    update = stream.pending.float()
+    if stream.pending_norm is not None:
+        weight, eps = stream.pending_norm
+        deviation = update - update.mean(dim=-1, keepdim=True)
+        update = deviation / torch.sqrt((deviation * deviation).mean(dim=-1, keepdim=True) + eps) * weight
+    return update
+
+
 def _hidden(stream: ResidualStream):
     """The hidden state as a value: the residual with its pending update added."""
     if stream.pending is None:
         return stream.residual.clone()
-    return stream.residual + stream.pending.float()
+    return stream.residual + _pending(stream)
 
 
 @register_part("block", "pre_norm")
@@ -146,13 +165,45 @@ class ParallelPreNormBlock(Block):
         ctx.trace("hidden_post_ffn", lambda: _hidden(stream))
 
 
+@register_part("block", "sandwich_norm")
+class SandwichNormBlock(Block):
+    sub_parts = (("mixer_norm", "norm"), ("mixer", "mixer"), ("mixer_output_norm", "norm"),
+                 ("feed_forward_norm", "norm"), ("feed_forward", "feed_forward"), ("feed_forward_output_norm", "norm"))
+    optional_parts = ("feed_forward_norm", "feed_forward", "feed_forward_output_norm")
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        for norm in (self.mixer_output_norm, self.feed_forward_output_norm):
+            if norm is not None and (norm.kind != "layernorm" or norm.bias_name):
+                raise ValueError("the sandwich_norm block norms a sublayer's output by a layernorm without a bias")
+
+    def forward(self, stream: ResidualStream, ctx: StepContext, cache: CacheHandle) -> None:
+        ctx.trace("hidden_in", lambda: _hidden(stream))
+        ctx.float_updates = True
+        try:
+            x = self.mixer_norm.forward(stream, ctx)
+            ctx.trace("normed", x)
+            stream.pending = self.mixer.forward(x, ctx, cache)
+            stream.pending_norm = (self.mixer_output_norm.weight, self.mixer_output_norm.eps)
+            ctx.trace("o", stream.pending)
+            if self.feed_forward is not None:
+                x = self.feed_forward_norm.forward(stream, ctx)
+                ctx.trace("mlp_input", x)
+                stream.pending = self.feed_forward.forward(x, ctx)
+                stream.pending_norm = (self.feed_forward_output_norm.weight, self.feed_forward_output_norm.eps)
+                ctx.trace("down", stream.pending)
+        finally:
+            ctx.float_updates = False
+        ctx.trace("hidden_post_ffn", lambda: _hidden(stream))
+
+
 def hidden_image(stream: ResidualStream, ctx: StepContext) -> torch.Tensor:
     """The hidden state in the compute dtype, for a part that reads it un-normed:
     the residual itself in float32, else its rounded image (made here if nobody
     left one).  A pending update is added first."""
     if stream.pending is not None:
-        stream.residual += stream.pending.float()
-        stream.pending, stream.image = None, None
+        stream.residual += _pending(stream)
+        stream.pending, stream.pending_norm, stream.image = None, None, None
     if ctx.rt.dtype == torch.float32:
         return stream.residual
     if stream.image is None:

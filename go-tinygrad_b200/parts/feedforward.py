@@ -8,7 +8,9 @@ up product's float sums, in its epilogue).  Parameters:
 
 ``swiglu``: dense gated feed-forward (SwiGLU): down(silu(gate(x)) * up(x)), silu(g) =
 g / (1 + exp(-g)) (model/llama.go:1361-1401, backends/simd/vec.go:52-59); with
-``activation`` "gelu_tanh" or "relu2" that function stands in silu's place on the gate.
+``activation`` "gelu_tanh" or "relu2" that function stands in silu's place on the gate.  With
+``gate_limit`` L the gated product is the clamped one: g = min(gate(x), L), u = up(x) between
+-L and L, g sigmoid(1.702 g) (u + 1) (`ops.ClampedGate`; not in the reference).
 
 Parameters: ``hidden_size``, ``intermediate_size`` and the tensor names
 ``gate``, ``up``, ``down``, and optionally ``gate_bias``, ``up_bias``,
@@ -39,7 +41,12 @@ ungated, down(act(up(x))) with ``activation`` ("relu2", "gelu_tanh", "silu");
 logit, not renormalised (the largest sigmoids are the largest logits);
 ``weight_on`` "input" multiplies the expert's input by the weight instead of
 its output: the update is the plain sum of expert(weight * x), the scaled rows
-formed in float and rounded once.  The reference has no routed feed-forward.
+formed in float and rounded once.  ``scoring`` "softmax_all": scores are the softmax over
+all the router's outputs, the largest score + ``correction`` (a tensor name) are chosen, and
+the weights are the chosen scores over their sum (+ 1e-20), times ``weight_scale``.
+``identity`` n: the router has n further outputs whose expert is the input itself, without
+tensors.  ``gate_limit`` as in ``swiglu``.  ``shared``: the spec of a feed-forward that every
+token passes beside its experts, added to their sum.  The reference has no routed feed-forward.
 """
 from __future__ import annotations
 
@@ -49,7 +56,7 @@ import torch
 
 from ..kernels import ops
 from ..weights.binder import WeightSpec
-from .base import FeedForward, Runtime, StepContext, emit_update, register_part, update_operand
+from .base import FeedForward, Runtime, StepContext, build_part, emit_update, register_part, update_operand
 
 
 @register_part("feed_forward", "swiglu")
@@ -62,8 +69,12 @@ class SwiGLU(FeedForward):
         self.activation = str(self.p.get("activation") or "silu")
         if self.activation not in ops.ACTIVATIONS:
             raise ValueError(f"feed-forward activation {self.activation!r} is not known; known: {sorted(ops.ACTIVATIONS)}")
+        limit = self.p.get("gate_limit")
+        self.gate = ops.ClampedGate(float(limit)) if limit is not None else None
+        if self.gate and self.activation != "silu":
+            raise ValueError("a clamped gate has an activation of its own")
         biases = [self.p.get(k) for k in ("gate_bias", "up_bias", "down_bias")]
-        if any(biases) and self.activation != "silu":
+        if any(biases) and (self.activation != "silu" or self.gate):
             raise ValueError("a gated feed-forward with biases uses the silu activation")
         if any(biases) and not all(biases):
             raise ValueError("a gated feed-forward has biases on all three projections or on none")
@@ -107,13 +118,13 @@ class SwiGLU(FeedForward):
             return self._forward_biased(x, ctx)
         act = update_operand(ctx, n, self.inter)
         if self.fused:
-            ops.linear(x, self.w_gate_up, act, epilogue=ops.GATED_EPILOGUES[self.activation])
+            ops.linear(x, self.w_gate_up, act, epilogue=self.gate or ops.GATED_EPILOGUES[self.activation])
         else:
             gate_up = rt.empty(n, 2 * self.inter)
             ops.linear(x, self.w_gate_up, gate_up)
             ctx.trace("gate_pre", gate_up[:, : self.inter])
             ctx.trace("up", gate_up[:, self.inter:])
-            ops.swiglu(gate_up, act, self.activation)
+            ops.swiglu(gate_up, act, self.gate or self.activation)
         ctx.trace("gate_act", act)
         return emit_update(act, self.w_down, ctx)
 
@@ -145,8 +156,10 @@ class RoutedExperts(FeedForward):
         self.inter = int(self.param("intermediate_size"))
         self.n_experts = int(self.param("n_experts"))
         self.top = int(self.param("top"))
-        if not 0 < self.top <= self.n_experts:
-            raise ValueError(f"a token cannot use {self.top} of {self.n_experts} experts")
+        self.n_identity = int(self.p.get("identity") or 0)
+        self.n_outputs = self.n_experts + self.n_identity
+        if not 0 < self.top <= self.n_outputs:
+            raise ValueError(f"a token cannot use {self.top} of {self.n_outputs} experts")
         self.gated = self.p.get("gate") is not None
         self.activation = str(self.p.get("activation") or ("silu" if self.gated else "relu2"))
         if self.gated and self.activation != "silu":
@@ -159,6 +172,21 @@ class RoutedExperts(FeedForward):
         self.weight_on = str(self.p.get("weight_on") or "output")
         if self.weight_on not in ("input", "output"):
             raise ValueError(f"an expert's weight multiplies its 'input' or its 'output', not {self.weight_on!r}")
+        limit = self.p.get("gate_limit")
+        self.gate = ops.ClampedGate(float(limit)) if limit is not None else "swiglu"
+        if limit is not None and not self.gated:
+            raise ValueError("a limit on the gate needs gated experts")
+        correction = self.p.get("correction")
+        self.correction_name = str(correction) if correction else None
+        self.weight_scale = float(self.p["weight_scale"]) if self.p.get("weight_scale") is not None else 1.0
+        if (correction or self.weight_scale != 1.0) and self.scoring != "softmax_all":
+            raise ValueError("a correction of the choice and a scale of the weights go with the scoring over all outputs")
+        if self.n_identity and (self.weight_on == "input" or not self.gated):
+            raise ValueError("identity experts are built beside gated experts weighted at their output")
+        shared = self.p.get("shared")
+        self.shared = build_part("feed_forward", shared) if shared is not None else None
+        if self.shared and (self.weight_on == "input" or not self.gated):
+            raise ValueError("a shared expert is built beside gated experts weighted at their output")
         self.matrices = ("gate", "up", "down") if self.gated else ("up", "down")
         self.names = {k: str(self.param(k)) for k in ("router",) + self.matrices}
         for k in self.matrices:
@@ -166,15 +194,20 @@ class RoutedExperts(FeedForward):
                 raise ValueError(f"the experts' tensor name {self.names[k]!r} needs '{{e}}' for the expert's index")
         bias = self.p.get("router_bias")
         self.router_bias_name = str(bias) if bias else None
-        self.router = self.router_bias = self.w_gate_up = self.w_down = None
+        self.router = self.router_bias = self.correction = self.w_gate_up = self.w_down = None
+
+    def children(self):
+        return [self.shared] if self.shared else []
 
     def _name(self, k: str, e: int) -> str:
         return self.names[k].replace("{e}", str(e))
 
     def weight_specs(self) -> List[WeightSpec]:
-        specs = [WeightSpec(self.names["router"], (self.n_experts, self.hidden))]
+        specs = [WeightSpec(self.names["router"], (self.n_outputs, self.hidden))]
         if self.router_bias_name:
-            specs.append(WeightSpec(self.router_bias_name, (self.n_experts,), role="parameter", std=0.02))
+            specs.append(WeightSpec(self.router_bias_name, (self.n_outputs,), role="parameter", std=0.02))
+        if self.correction_name:
+            specs.append(WeightSpec(self.correction_name, (self.n_outputs,), role="parameter", std=0.02))
         for e in range(self.n_experts):
             if self.gated:
                 specs.append(WeightSpec(self._name("gate", e), (self.inter, self.hidden)))
@@ -185,6 +218,7 @@ class RoutedExperts(FeedForward):
     def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
         self.router = rt.vector(tensors[self.names["router"]])
         self.router_bias = rt.vector(tensors[self.router_bias_name]) if self.router_bias_name else None
+        self.correction = rt.vector(tensors[self.correction_name]) if self.correction_name else None
         # [E, 2I, H]: an expert's gate rows, then its up rows -- or, where the products run on the
         # tensor cores and apply the gated silu in their epilogue, alternating in blocks of 8; [E, H, I]
         self.fused = rt.dtype == torch.bfloat16 and self.inter % 8 == 0 and self.hidden % 8 == 0
@@ -203,7 +237,7 @@ class RoutedExperts(FeedForward):
         n, top, E = x.shape[0], self.top, self.n_experts
         chosen = rt.empty(n, top, dtype=torch.int32)
         weights = rt.empty(n, top, dtype=torch.float32)
-        ops.moe_route(x, self.router, self.router_bias, chosen, weights, self.scoring)
+        ops.moe_route(x, self.router, self.router_bias, chosen, weights, self.scoring, self.correction, self.weight_scale)
         ctx.trace("experts", chosen)
         if not self.gated or self.weight_on == "input":
             return self._forward_general(x, ctx, chosen, weights)
@@ -221,18 +255,28 @@ class RoutedExperts(FeedForward):
             # prompt-sized: the inputs copied into arranged order, for the product that tensor copies feed
             gathered = rt.empty(rows, self.hidden)
             ops.moe_gather(x, row_item, top, gathered)
-            ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, act, epilogue="swiglu")
+            ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, act, epilogue=self.gate)
         elif fused:
-            ops.moe_product(x, row_item, top, self.w_gate_up, tile_expert, act, epilogue="swiglu")
+            ops.moe_product(x, row_item, top, self.w_gate_up, tile_expert, act, epilogue=self.gate)
         else:
             sums = rt.empty(rows, 2 * self.inter, dtype=torch.float32)
             ops.moe_product(x, row_item, top, self.w_gate_up, tile_expert, sums)
-            ops.swiglu_bias(sums, None, None, act)
+            ops.swiglu_bias(sums, None, None, act, epilogue=self.gate)
         y = rt.empty(rows, self.hidden, dtype=torch.float32)
         ops.moe_product(act, row_item, 0, self.w_down, tile_expert, y)
         out = rt.empty(n, self.hidden, dtype=torch.float32 if ctx.float_updates else None)
-        ops.moe_combine(y, item_row, weights, out)
+        ops.moe_combine(y, item_row, weights, out, x=x if self.n_identity else None, base=self._shared_update(x, ctx))
         return out
+
+    def _shared_update(self, x: torch.Tensor, ctx: StepContext) -> Optional[torch.Tensor]:
+        """The shared expert's update in float32; None without one, or where it has joined the residual already."""
+        if self.shared is None:
+            return None
+        before, ctx.float_updates = ctx.float_updates, True
+        try:
+            return self.shared.forward(x, ctx)
+        finally:
+            ctx.float_updates = before
 
 
     def _forward_general(self, x: torch.Tensor, ctx: StepContext, chosen: torch.Tensor, weights: torch.Tensor) -> torch.Tensor:
@@ -254,11 +298,11 @@ class RoutedExperts(FeedForward):
         ops.moe_gather(x, row_item, top, gathered, weights=weights if on_input else None)
         act = rt.empty(rows, self.inter)
         if self.gated and fused:
-            ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, act, epilogue="swiglu")
+            ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, act, epilogue=self.gate)
         elif self.gated:
             sums = rt.empty(rows, 2 * self.inter, dtype=torch.float32)
             ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, sums)
-            ops.swiglu_bias(sums, None, None, act)
+            ops.swiglu_bias(sums, None, None, act, epilogue=self.gate)
         else:
             ops.moe_product(gathered, row_item, 0, self.w_gate_up, tile_expert, act, epilogue=self.activation)
         ctx.trace("gate_act", act)

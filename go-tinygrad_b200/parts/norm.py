@@ -13,7 +13,9 @@ update by its links on the way.
 ``layernorm``: y = (x - mean(x)) / sqrt(var(x) + eps) * w + b, var the mean of
 the squared deviations, all in float32.  Parameters: ``size``, ``eps``,
 ``weight`` and ``bias`` (tensor names; ``bias`` None for a norm without one).
-The reference has no such norm.
+The reference has no such norm.  Handed a stream whose pending update has a norm of its
+own to pass (`ResidualStream.pending_norm`), it norms the update, adds it and norms
+the sum in one pass.
 """
 from __future__ import annotations
 
@@ -66,6 +68,8 @@ class RMSNorm(Norm):
             if rows is None:
                 stream.pending, stream.pending_links, stream.image = None, None, None
             return out
+        if stream.pending_norm is not None:
+            raise ValueError("an update that passes a layer norm before it is added can only be followed by a layer norm")
         ops.add_rmsnorm(stream.residual, stream.pending, self.weight, self.eps, out, rows)
         if rows is None:
             if stream.pending is not None:
@@ -100,9 +104,12 @@ class LayerNorm(Norm):
                 rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         n_out = rows.numel() if rows is not None else stream.residual.shape[0]
         out = ctx.rt.empty(n_out, self.size)
-        ops.add_layernorm(stream.residual, stream.pending, self.weight, self.bias, self.eps, out, rows)
+        if stream.pending is not None and stream.pending_norm is not None:
+            ops.layernorm_add_layernorm(stream.residual, stream.pending, *stream.pending_norm, self.weight, self.bias, self.eps, out, rows)
+        else:
+            ops.add_layernorm(stream.residual, stream.pending, self.weight, self.bias, self.eps, out, rows)
         if rows is None:
             if stream.pending is not None:
                 stream.image = None
-            stream.pending = None
+            stream.pending, stream.pending_norm = None, None
         return out

@@ -28,6 +28,9 @@ and the frequency is f_i (1 - r_i) + f_i / factor * r_i.  Cosines and sines
 are multiplied by 0.1 ln(factor) + 1, which sharpens the attention as the
 context is stretched.
 
+The linear scaling (``scaling`` = {"rope_type": "linear", factor}; not in the
+reference) divides every frequency by `factor`.
+
 ``sinusoidal``: absolute positions, added to the embedded tokens: channel 2i gets
 sin(p f_i), channel 2i+1 cos(p f_i), f_i = base^(-2i/size).  Queries and keys are
 not rotated.  Parameters: ``size`` (of the hidden state), ``base``.  The embedding
@@ -71,6 +74,8 @@ def rotary_frequencies(head_dim: int, theta: float, scaling: Optional[Mapping] =
         factor = float(scaling["factor"])
         ramp = yarn_ramp(head_dim, theta, float(scaling["original"]), float(scaling["fast"]), float(scaling["slow"]))
         return [f / factor * r + f * (1.0 - r) for f, r in zip(freqs, ramp)]
+    if scaling and scaling.get("rope_type") == "linear":
+        return [f / float(scaling["factor"]) for f in freqs]
     if scaling:
         factor = float(scaling["factor"])
         low = float(scaling["low_freq_factor"])

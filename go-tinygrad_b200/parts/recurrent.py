@@ -471,3 +471,79 @@ class MatrixMemory(Mixer):
         ops.head_norm_gate(num, proj[:, 2 * a + self.v_width: 2 * (a + self.v_width)], self.norm_w, self.eps, out, h, den=den)
         ctx.trace("attn", out)
         return emit_update(out, self.w_o, ctx)
+
+
+@register_part("mixer", "lightning")
+class Lightning(Mixer):
+    """Linear attention with a fixed decay per head (lightning attention).
+
+    q = silu(W_q x) and k = silu(W_k x) (``n_heads`` heads of ``head_dim``), v = silu(W_v x)
+    (heads of ``value_dim``).  Per head, token by token, with its number a of ``decay``,
+
+        S <- a S + k v^T;  o = S^T q        (S: head_dim x value_dim, zero at the start)
+
+    The concatenated heads are divided by their common root mean square (``eps``),
+    multiplied by a weight of all heads' channels and by sigmoid(W_g x), and projected by
+    W_o.  What a sequence keeps between steps is S, a float32 `StateRequest`.  The state,
+    the decays, the sums and the norm are float32 in both compute dtypes; the projections
+    with their activations are in the compute dtype.  The reference has no recurrent mixer.
+
+    Parameters: ``hidden_size``, ``n_heads``, ``head_dim``, ``value_dim``, ``decay`` (one
+    number a head), ``eps`` and the tensor names ``q``, ``k``, ``v``, ``g``, ``norm``, ``o``.
+    """
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden = int(self.param("hidden_size"))
+        self.n_heads = int(self.param("n_heads"))
+        self.dim = int(self.param("head_dim"))
+        self.vdim = int(self.param("value_dim"))
+        self.eps = float(self.param("eps"))
+        self.decays = [float(a) for a in self.param("decay")]
+        if len(self.decays) != self.n_heads:
+            raise ValueError(f"{self.n_heads} heads need as many decays, not {len(self.decays)}")
+        if self.dim > ops.LIGHTNING_MAX_KEY_DIM:
+            raise ValueError(f"heads of {self.dim} key channels are more than the recurrence's kernel takes ({ops.LIGHTNING_MAX_KEY_DIM})")
+        self.names = {k: str(self.param(k)) for k in ("q", "k", "v", "g", "norm", "o")}
+        self.qk_width, self.v_width = self.n_heads * self.dim, self.n_heads * self.vdim
+        self.w_qkv: Optional[torch.Tensor] = None
+
+    def weight_specs(self) -> List[WeightSpec]:
+        n = self.names
+        return [WeightSpec(n["q"], (self.qk_width, self.hidden)), WeightSpec(n["k"], (self.qk_width, self.hidden)),
+                WeightSpec(n["v"], (self.v_width, self.hidden)), WeightSpec(n["g"], (self.v_width, self.hidden)),
+                WeightSpec(n["norm"], (self.v_width,), role="vector", mean=1.0), WeightSpec(n["o"], (self.hidden, self.v_width))]
+
+    def cache_requests(self) -> List[Request]:
+        return [StateRequest("memory", (self.n_heads, self.dim, self.vdim), "float32")]
+
+    def last_product(self):
+        return self.names["o"], self.v_width
+
+    def load(self, tensors: Mapping[str, torch.Tensor], rt: Runtime) -> None:
+        n = self.names
+        self.w_qkv = rt.matrix(torch.cat([tensors[n[k]].to(rt.dtype) for k in ("q", "k", "v")], dim=0))
+        self.w_g = rt.matrix(tensors[n["g"]])
+        self.norm_w = rt.vector(tensors[n["norm"]])
+        self.decay = rt.vector(torch.tensor(self.decays, dtype=torch.float64))
+        if not self.joined:
+            self.w_o = rt.matrix(tensors[n["o"]])
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheHandle) -> torch.Tensor:
+        rt, n, a = ctx.rt, x.shape[0], self.qk_width
+        if not cache.writes:
+            raise ValueError("a recurrent mixer cannot read another run's state: every run advances its own")
+        padded = lambda width: (width + 7) // 8 * 8
+        width = 2 * a + self.v_width
+        qkv = rt.empty(n, padded(width))[:, : width]
+        ops.linear(x, self.w_qkv, qkv, epilogue="silu")
+        gate = rt.empty(n, padded(self.v_width))[:, : self.v_width]
+        ops.linear(x, self.w_g, gate)
+        y = rt.empty(n, padded(self.v_width), dtype=torch.float32)[:, : self.v_width]
+        ops.lightning_scan(qkv[:, :a], qkv[:, a: 2 * a], qkv[:, 2 * a:], self.decay, cache.state("memory"), y, ctx.cu_seqlens, ctx.slots,
+                           ctx.n_seqs, one_token_each=ctx.is_decode)
+        ctx.trace("scan", y)
+        out = update_operand(ctx, n, self.v_width)
+        ops.head_norm_gate(y, gate, self.norm_w, self.eps, out, 1)
+        ctx.trace("attn", out)
+        return emit_update(out, self.w_o, ctx)
