@@ -910,11 +910,11 @@ LIGHTNING_MAX_KEY_DIM = 512   # most key channels a head of linear attention may
 
 
 def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
-                   cu_seqlens, slots, n_seqs: int, one_token_each: bool = False) -> None:
+                   ctx) -> None:
     """Linear attention with a fixed decay per head (csrc/lightning.cu): S <- decay S + k v^T, out = S^T q;
     q, k [n, heads * d] and v [n, heads * dv], columns of one matrix; decay float32 [heads]; state float32
-    [slots, heads, d, dv], read and left per sequence; out float32 [n, heads * dv].  `one_token_each`: row
-    b is sequence b's only token."""
+    [slots, heads, d, dv], read and left per sequence; out float32 [n, heads * dv].  `ctx`: the step's
+    context (rows, sequences, slots)."""
     for name, t in (("q", q), ("k", k), ("v", v), ("out", out)):
         _rows2d(t, f"lightning_scan: {name}")
     heads = decay.numel()
@@ -926,12 +926,11 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     _need(out.dtype == torch.float32 and tuple(out.shape) == (n, heads * dv), "lightning_scan: out must be float32 [n, heads * dv]")
     _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, d, dv), "lightning_scan: state must be float32 [slots, heads, d, dv]")
     _need(d <= LIGHTNING_MAX_KEY_DIM, f"lightning_scan: heads of {d} key channels exceed {LIGHTNING_MAX_KEY_DIM}")
-    _int32("lightning_scan", cu_seqlens, slots)
-    if one_token_each:
-        _need(n == n_seqs, "lightning_scan: one token each means as many rows as sequences")
+    _int32("lightning_scan", ctx.cu_seqlens, ctx.slots)
+    _need(n == ctx.n_tokens, "lightning_scan: as many rows as the step has tokens")
     _check(_fn("gtg_lightning_scan")(_dt(q), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), _ptr(state), _ptr(out), out.stride(0),
-                                     _ptr(cu_seqlens), _ptr(slots), int(n_seqs), heads, d, dv, 1 if one_token_each else 0, _stream()),
-           "lightning_scan")
+                                     _ptr(ctx.cu_seqlens), _ptr(ctx.slots), int(ctx.n_seqs), heads, d, dv, 1 if ctx.is_decode else 0,
+                                     _stream()), "lightning_scan")
 
 
 # ------------------------------------------------------------- recurrent mixers

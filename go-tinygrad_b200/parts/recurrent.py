@@ -540,8 +540,7 @@ class Lightning(Mixer):
         gate = rt.empty(n, padded(self.v_width))[:, : self.v_width]
         ops.linear(x, self.w_g, gate)
         y = rt.empty(n, padded(self.v_width), dtype=torch.float32)[:, : self.v_width]
-        ops.lightning_scan(qkv[:, :a], qkv[:, a: 2 * a], qkv[:, 2 * a:], self.decay, cache.state("memory"), y, ctx.cu_seqlens, ctx.slots,
-                           ctx.n_seqs, one_token_each=ctx.is_decode)
+        ops.lightning_scan(qkv[:, :a], qkv[:, a: 2 * a], qkv[:, 2 * a:], self.decay, cache.state("memory"), y, ctx)
         ctx.trace("scan", y)
         out = update_operand(ctx, n, self.v_width)
         ops.head_norm_gate(y, gate, self.norm_w, self.eps, out, 1)

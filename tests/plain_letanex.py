@@ -179,22 +179,28 @@ def clamped_expert(h, gate, up, down, limit):
     return (g * sigmoid(1.702 * g) * (u + 1.0)) @ A(down).T
 
 
-def route(h, router, correction, top, scale):
-    """(chosen [T, top], weights [T, top]): softmax scores over all outputs; the
-    largest scores plus correction choose; the weights are the chosen scores
-    without it, over their sum, times scale."""
+def scores(h, router):
     z = h @ A(router).T
     s = np.exp(z - z.max(axis=-1, keepdims=True))
-    s = s / s.sum(axis=-1, keepdims=True)
-    chosen = np.argsort(-(s + A(correction)), axis=-1, kind="stable")[:, :top]
+    return s / s.sum(axis=-1, keepdims=True)
+
+
+def route(h, router, correction, top, scale, chosen=None):
+    """(chosen [T, top], weights [T, top]): softmax scores over all outputs; the
+    largest scores plus correction choose; the weights are the chosen scores
+    without it, over their sum, times scale.  `chosen`: take these choices instead (of a
+    run whose rounding may have turned a close call)."""
+    s = scores(h, router)
+    if chosen is None:
+        chosen = np.argsort(-(s + A(correction)), axis=-1, kind="stable")[:, :top]
     w = np.take_along_axis(s, chosen, axis=-1)
     return chosen, w / (w.sum(axis=-1, keepdims=True) + 1e-20) * scale
 
 
-def mixture(h, W, p, mlp):
+def mixture(h, W, p, mlp, chosen=None):
     """`W`: every tensor by its full name; `p`: the feed-forward's prefix."""
     r = mlp["router"]
-    chosen, weights = route(h, W[p + "router"], W[p + "correction"], r["top"], r["scale"])
+    chosen, weights = route(h, W[p + "router"], W[p + "correction"], r["top"], r["scale"], chosen)
     out = np.zeros_like(h)
     for t in range(h.shape[0]):
         for e, w in zip(chosen[t], weights[t]):
@@ -212,12 +218,14 @@ def mixture(h, W, p, mlp):
 # --------------------------------------------------------------------------
 # the whole model
 # --------------------------------------------------------------------------
-def forward(cfg, W, tokens, layers_out=None):
+def forward(cfg, W, tokens, layers_out=None, choices=None, slack=None):
     """Logits [T, vocab] of one sequence.  `W`: every tensor by its full name;
-    `layers_out`, a list, receives the hidden state after every layer."""
+    `layers_out`, a list, receives the hidden state after every layer.  `choices`: the experts
+    to use per mixture, in order ([T, top] each), in place of those the scores choose; `slack`,
+    a list, then receives by how much each such choice was worse than the best."""
     eps = float(cfg["norm"]["eps"])
     x = A(W["embed"])[np.asarray(tokens)]
-    cached = {}
+    cached, choices = {}, iter(choices) if choices is not None else None
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
         m = layer["mixer"]
@@ -237,7 +245,12 @@ def forward(cfg, W, tokens, layers_out=None):
             if mlp["kind"] == "dense":
                 update = squared_relu(h, W[p + "mlp.up"], W[p + "mlp.down"])
             else:
-                update = mixture(h, W, p + "mlp.", mlp)
+                chosen = next(choices) if choices is not None else None
+                if slack is not None:
+                    s = scores(h, W[p + "mlp.router"]) + A(W[p + "mlp.correction"])
+                    best = -np.sort(-s, axis=-1)[:, :chosen.shape[1]].sum(axis=-1)
+                    slack.append(best - np.take_along_axis(s, chosen, axis=-1).sum(axis=-1))
+                update = mixture(h, W, p + "mlp.", mlp, chosen)
             x = x + layer_norm(update, W[p + "norm2b"], eps)
         if layers_out is not None:
             layers_out.append(x.copy())
