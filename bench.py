@@ -41,8 +41,11 @@ a gate on all channels, attention through a latent with sinks, the gated delta
 rule; see `megerax_shape`), and with --design mererax for the Mererax design
 (mixer and feed-forward side by side, the selective scan, attention with a
 penalty on the distance beside a matrix memory; see `mererax_shape`), which also
-measures the Ropovik design, the closest other one, beside it.  The default run
-is not changed by any of them.
+measures the Ropovik design, the closest other one, beside it, and with --design
+letanex for the Letanex design (differential attention, linear attention with a
+fixed decay per head, mixtures with identities and a shared expert; see
+`letanex_shape`), beside which the Zotolix design, the closest other one, is
+measured.  The default run is not changed by any of them.
 
 Peaks come from MEASURED_PEAKS.json beside this file if present, else from the
 fallback figures of an earlier measurement on the same pool.  Inputs are larger
@@ -541,6 +544,23 @@ def mererax_shape(width, heads, kv_heads, dim, ff, inner, state, rank, m_heads, 
             "layers": [scan, pair] * 4}
 
 
+def letanex_shape(width, heads, kv_heads, ff, experts, expert_ff, top, vocab=32000):
+    """Eight layers, linear attention (heads of 128 x 128) and differential attention (two maps of 64 channels over values of
+    128) in turn, every second attention layer reading the keys of the one before; the first layer's feed-forward is
+    dense, the others' are mixtures of `experts` experts and four identities (`top` to a token) beside a shared expert."""
+    decay = [round(1.0 - 2.0 ** (-1.0 - 9.0 * (i + 1) / (width // 128)), 6) for i in range(width // 128)]
+    light = {"heads": width // 128, "dim": 128, "vdim": 128, "decay": decay}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
+           "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 4.0}}}
+    routed = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "shared": {"ff": expert_ff, "limit": 7.0},
+              "router": {"experts": experts, "top": top, "identity": 4, "scale": 1.5}}
+    layers = []
+    for i in range(8):
+        mixer = light if i % 2 == 0 else dict(att, kv_from=i - 2) if i % 4 == 3 else att
+        layers.append({"type": "attention" if i % 2 else "lightning", "mixer": mixer, "mlp": routed if i else {"kind": "dense", "ff": ff}})
+    return {"architecture": "Letanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 DESIGN_SIZES = {
     # the layer sizes of Llama-3.2-1B / SmolLM2 (width 2048) and of Llama-3.1-8B (width 4096); the
     # recurrence has twice the width in its inner size, heads of 64 and a state of 128, as Mamba-2 models do
@@ -575,7 +595,18 @@ MERERAX_SIZES = {
     "w4096": (mererax_shape(4096, 32, 8, 128, 14336, 8192, 16, 256, 8, 256, 512), dict(LLAMA_3P1_8B, num_hidden_layers=8, vocab_size=32000),
               DESIGN_SIZES["w4096"][0]),
 }
+LETANEX_SIZES = {
+    # the same two widths; queries, values and outputs as wide as the model, a quarter as many key heads as query heads; 16
+    # experts of a quarter of the dense feed-forward's size, four to a token; the third is the Zotolix design at equal size
+    "w2048": (letanex_shape(2048, 16, 4, 8192, 16, 2048, 4), dict(LLAMA_3P2_1B, num_hidden_layers=8, vocab_size=32000), ZOTOLIX_SIZES["w2048"][0]),
+    "w4096": (letanex_shape(4096, 32, 8, 14336, 16, 3584, 4), dict(LLAMA_3P1_8B, num_hidden_layers=8, vocab_size=32000), ZOTOLIX_SIZES["w4096"][0]),
+}
 DESIGNS = {
+    "letanex": (LETANEX_SIZES, "8 layers, linear attention (heads of 128 x 128) and differential attention (two maps of 64 channels over values "
+                               "of 128, every second such layer reading the keys of the one before) in turn, each sublayer between two "
+                               "layer norms; one dense squared-relu feed-forward, then mixtures of 16 experts with clamped gates and 4 "
+                               "identities (4 to a token) beside a shared expert; beside 8 Llama layers of equal width and the Zotolix "
+                               "design (attention and mixtures of 16 experts); vocabulary 32000"),
     "mererax": (MERERAX_SIZES, "8 layers, a selective scan (16 states a channel) and a pair of mixers (attention with a penalty on the "
                                "distance whose values are the keys, beside a matrix memory of eight heads) in turn, a gated silu "
                                "feed-forward beside each mixer; beside 8 Llama layers of equal width, heads and feed-forward size and "
@@ -1214,13 +1245,148 @@ def run_design(args):
                 n * inner * (4 + 2 + 2))
         return rows
 
+    def letanex_kernel_table(cfg):
+        """Each kernel the Letanex design added or extended, alone, at this size: a prompt of T tokens and a
+        decode step of 64 sequences after 1,024 tokens; the bytes it has to move against the copy peak and,
+        for products and attention, its FLOPs against the matrix peak.  Beside each the like kernel of the
+        Llama, Ropovik, Mererax or Zotolix path at the same rows."""
+        from go_tinygrad_b200.cache import Cache, KVRequest
+        from go_tinygrad_b200.parts.base import StepContext
+        bf, f32, i32 = torch.bfloat16, torch.float32, torch.int32
+        li, a, mx = cfg["layers"][0]["mixer"], cfg["layers"][1]["mixer"], cfg["layers"][1]["mlp"]
+        H, heads, n_kv, d, vd = cfg["width"], a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        E, idn, top, eff = mx["router"]["experts"], mx["router"]["identity"], mx["router"]["top"], mx["expert"]["ff"]
+        lh, ld, lv = li["heads"], li["dim"], li["vdim"]
+        rows = []
+
+        def add(name, rows_n, ms, nbytes, flops=0, like=None):
+            rows.append({"kernel": name, "rows": rows_n, "us": round(ms * 1e3, 2), "mb": round(nbytes / 1e6, 2),
+                         "of_copy_peak": round(nbytes / ms / 1e6 / pk["hbm_gbs"], 3),
+                         **({"tflops": round(flops / ms / 1e9, 1), "of_matrix_peak": round(flops / ms / 1e9 / pk["bf16_tflops"], 3)} if flops else {}),
+                         **({"like": like} if like else {})})
+        rnd = lambda *shape, dtype=bf: torch.randn(*shape, device=dev, dtype=f32).to(dtype)
+        for n, n_seqs, ctx_len, tag in ((T, 1, 0, "prompt"), (64, 64, prompt_len, "decode")):
+            per = n // n_seqs
+            one = per == 1
+            rt = lib.parts.Runtime(dev, bf)
+            cache = Cache([[KVRequest(n_kv, 2 * d, None, value_dim=vd)], [KVRequest(2 * n_kv, d, None)]], [None, None],
+                          max_tokens=64 * ((ctx_len + per + 63) // 64) * n_seqs, max_slots=n_seqs, dtype=bf, device=dev)
+            slot_list = [cache.open_sequence() for _ in range(n_seqs)]
+            cache.reserve_many([(s, ctx_len + per) for s in slot_list]); cache.flush_tables()
+            for g in cache.groups:
+                g.storage.normal_()
+            kv, kv_like = cache.handles[0].kv, cache.handles[1].kv
+            cu = torch.arange(0, n + 1, per, dtype=i32, device=dev)
+            seq = torch.arange(n, dtype=i32, device=dev) // per
+            slots = torch.tensor(slot_list, dtype=i32, device=dev)
+            start = torch.full((n_seqs,), ctx_len, dtype=i32, device=dev)
+            pos = (start[seq.long()] + (torch.arange(n, device=dev) % per)).to(i32)
+            ctx = StepContext(rt=rt, n_tokens=n, n_seqs=n_seqs, tokens=seq, positions=pos, token_seq=seq, cu_seqlens=cu, slots=slots,
+                              start_pos=start, max_q_len=per, max_kv_len=ctx_len + per, is_decode=one, total_kv_len=n_seqs * (ctx_len + per))
+            # the normed update joins the hidden state, which is normed again; beside the plain addition and norm
+            res, upd, w = rnd(n, H, dtype=f32), rnd(n, H, dtype=f32), rnd(H, dtype=f32)
+            upd16, out = upd.to(bf), torch.empty(n, H, dtype=bf, device=dev)
+            add(f"layernorm_add_layernorm ({tag})", n, timed(lambda: ops.layernorm_add_layernorm(res, upd, w, 1e-5, w, None, 1e-5, out)), n * H * (4 + 4 + 4 + 2))
+            add(f"add_layernorm ({tag})", n, timed(lambda: ops.add_layernorm(res, upd16, w, None, 1e-5, out)), n * H * (4 + 4 + 2 + 2), like="layernorm_add_layernorm")
+            # rotation of both maps and cache store, beside one map of twice the heads
+            C = heads * 2 * d + n_kv * (2 * d + vd)
+            sums, cs, q = rnd(n, C, dtype=f32), rnd(n, d // 2, 2, dtype=f32), torch.empty(n, heads * 2 * d, dtype=bf, device=dev)
+            add(f"qkv_finish, two maps ({tag})", n, timed(lambda: ops.qkv_finish(sums, None, cs, heads, kv, q, seq, slots, pos, maps=2)), n * C * 6)
+            add(f"qkv_finish ({tag})", n, timed(lambda: ops.qkv_finish(sums, None, cs, 2 * heads, kv_like, q, seq, slots, pos)), n * C * 6, like="qkv_finish, two maps")
+            # differential attention, beside ordinary heads of one map's size (half as wide values)
+            q.copy_(rnd(n, heads * 2 * d))
+            mixed = torch.empty(n, heads * vd, dtype=bf, device=dev)
+            keys = n_seqs * (ctx_len + 1) if one else per * (per + 1) // 2
+            add(f"attention_diff ({tag})", n, timed(lambda: ops.attention_diff(q, mixed, kv, ctx, heads, 0.125, 0.5, 0.5, 1e-5)),
+                n * heads * (2 * d + vd) * 2 + n_seqs * n_kv * (ctx_len + per) * (2 * d + vd) * 2, 4 * heads * keys * (d + vd))
+            nbytes = n * 2 * heads * d * 4 + n_seqs * 2 * n_kv * (ctx_len + per) * d * 4
+            if one:
+                splits, chunk, ring = ops.attention_decode_plan(n, 2 * heads, 2 * n_kv, d, ctx_len + 1, 0, n * (ctx_len + 1))
+                scratch = torch.empty(max(1, ops.attention_decode_scratch_floats(n, 2 * heads, d, splits)), dtype=f32, device=dev)
+                add(f"split-KV decode attention ({tag})", n,
+                    timed(lambda: ops.attention_decode_bf16(q, mixed, kv_like, slots, pos, 2 * heads, 0.125, 0, splits, scratch, chunk_pages=chunk, ring_pages=ring)),
+                    nbytes, 8 * heads * keys * d, like="attention_diff")
+                add(f"attention_general, warp-level ({tag})", n, timed(lambda: ops.attention_general(q, mixed, kv_like, ctx, 2 * heads, 0.125)),
+                    nbytes, 8 * heads * keys * d, like="attention_diff")
+            else:
+                add(f"attention, tcgen05 ({tag})", n,
+                    timed(lambda: ops.attention_prefill_tcgen05(q, mixed, kv_like, cu, slots, start, n_seqs, per, 2 * heads, 0.125)),
+                    nbytes, 8 * heads * keys * d, like="attention_diff")
+            # linear attention, beside the recurrences of the Ropovik and Mererax paths at as many state numbers
+            lw, vw = lh * ld, lh * lv
+            qkv, gate, dec = rnd(n, 2 * lw + vw), rnd(n, vw), torch.tensor(li["decay"], device=dev)
+            st, y = torch.zeros(n_seqs, lh, ld, lv, device=dev), torch.empty(n, vw, dtype=f32, device=dev)
+            add(f"lightning_scan ({tag})", n, timed(lambda: ops.lightning_scan(qkv[:, :lw], qkv[:, lw:2 * lw], qkv[:, 2 * lw:], dec, st, y, ctx)),
+                n * (2 * lw * 2 + vw * (2 + 4)) + n_seqs * lh * ld * lv * 8, 4 * n * lh * ld * lv)
+            sh, sp, sn, sg = lh * ld * lv // (64 * 128), 64, 128, 8
+            xs, bc = rnd(n, sh * sp), rnd(n, sg * sn, 2, dtype=f32)
+            dt_raw, dtb, alog, skip = rnd(n, sh), rnd(sh, dtype=f32), rnd(sh, dtype=f32), rnd(sh, dtype=f32)
+            S2, y2 = torch.zeros(n_seqs, sh, sn, sp, device=dev), torch.empty(n, sh * sp, dtype=f32, device=dev)
+            add(f"ssm_scan, as many state numbers ({tag})", n,
+                timed(lambda: ops.ssm_scan(xs, bc, dt_raw, dtb, alog, skip, S2, y2, cu, slots, n_seqs, sh, sg, sn, sp, one_token_each=one)),
+                n * (sh * sp * 6 + sg * sn * 8) + n_seqs * sh * sn * sp * 8, 4 * n * lh * ld * lv, like="lightning_scan")
+            gates, gb = rnd(n, 2 * lh, dtype=f32), torch.zeros(2 * lh, device=dev)
+            ms_st = (torch.zeros(n_seqs, lh, ld, lv, device=dev), torch.zeros(n_seqs, lh, ld, device=dev), torch.zeros(n_seqs, lh, lv + 1, device=dev))
+            den = torch.empty(n, lh, dtype=f32, device=dev)
+            add(f"mlstm_scan ({tag})", n,
+                timed(lambda: ops.mlstm_scan(qkv[:, :lw], qkv[:, lw:2 * lw], qkv[:, 2 * lw:], gates, gb, 15.0, ld ** -0.5, ms_st, y, den, cu, slots, n_seqs,
+                                             lh, one_token_each=one)),
+                n * (2 * lw * 2 + vw * (2 + 4) + 3 * lh * 4) + n_seqs * lh * ld * lv * 8, 4 * n * lh * ld * lv, like="lightning_scan")
+            nw, og = rnd(vw, dtype=f32), torch.empty(n, vw, dtype=bf, device=dev)
+            add(f"head_norm_gate, a row as one head ({tag})", n, timed(lambda: ops.head_norm_gate(y, gate, nw, 1e-5, og, 1)), n * vw * (4 + 2 + 2))
+            add(f"head_norm_gate ({tag})", n, timed(lambda: ops.head_norm_gate(y, gate, nw, 1e-5, og, lh)), n * vw * (4 + 2 + 2), like="head_norm_gate, a row as one head")
+            # the mixture: router, order, products, sum
+            x = rnd(n, H)
+            router, corr = rnd(E + idn, H, dtype=f32), torch.zeros(E + idn, device=dev)
+            chosen, weights = torch.empty(n, top, dtype=i32, device=dev), torch.empty(n, top, dtype=f32, device=dev)
+            add(f"moe_route, scores over all ({tag})", n, timed(lambda: ops.moe_route(x, router, None, chosen, weights, "softmax_all", corr, 1.5)),
+                n * (H * 2 + top * 8) + (E + idn) * H * 4)
+            plain, chosen2 = router[:E].contiguous(), torch.empty(n, top, dtype=i32, device=dev)
+            add(f"moe_route, sigmoid ({tag})", n, timed(lambda: ops.moe_route(x, plain, None, chosen2, weights, "sigmoid")),
+                n * (H * 2 + top * 8) + E * H * 4, like="moe_route, scores over all")
+            w_gu, w_dn = rnd(E, 2 * eff, H) * 0.02, rnd(E, H, eff) * 0.02
+            for label, ch, gate_e in (("", chosen, ops.ClampedGate(7.0)), (" silu", chosen2, "swiglu")):
+                tile = 128 if n * top >= 128 * E else ops.MOE_TILE_ROWS
+                tiles = ops.moe_tiles_cap(n * top, E, tile)
+                row_item, item_row = torch.empty(tiles * tile, dtype=i32, device=dev), torch.empty(n * top, dtype=i32, device=dev)
+                tile_e = torch.empty(tiles, dtype=i32, device=dev)
+                like = None if not label else "moe "
+                add(f"moe_arrange{label} ({tag})", n, timed(lambda: ops.moe_arrange(ch, E, row_item, item_row, tile_e, tile)), n * top * 12 + tiles * (tile + 1) * 4,
+                    like=like and "moe_arrange")
+                real = int((item_row >= 0).sum())
+                act, yy = torch.empty(tiles * tile, eff, dtype=bf, device=dev), torch.empty(tiles * tile, H, dtype=f32, device=dev)
+                gathered = torch.empty(tiles * tile, H, dtype=bf, device=dev)
+                used = int(torch.unique(ch[ch < E]).numel())
+                if tile == 128:
+                    ops.moe_gather(x, row_item, top, gathered)
+                    up = lambda: ops.moe_product(gathered, row_item, 0, w_gu, tile_e, act, epilogue=gate_e)
+                else:
+                    up = lambda: ops.moe_product(x, row_item, top, w_gu, tile_e, act, epilogue=gate_e)
+                add(f"moe gate/up product{label} ({tag})", n, timed(up), used * 2 * eff * H * 2 + real * (H + eff) * 2, 4 * real * H * eff,
+                    like=like and "moe gate/up product")
+                if not label:
+                    base, comb = rnd(n, H, dtype=f32), torch.empty(n, H, dtype=f32, device=dev)
+                    ops.moe_product(act, row_item, 0, w_dn, tile_e, yy)
+                    add(f"moe_combine, identities and shared ({tag})", n, timed(lambda: ops.moe_combine(yy, item_row, weights, comb, x=x, base=base)),
+                        real * H * 4 + (n * top - real) * H * 2 + n * H * 8)
+                else:
+                    add(f"moe_combine ({tag})", n, timed(lambda: ops.moe_combine(yy, item_row, weights, comb)), real * H * 4 + n * H * 4,
+                        like="moe_combine, identities and shared")
+                del act, yy, gathered
+            w_sh, act = rnd(2 * eff, H) * 0.02, torch.empty(n, eff, dtype=bf, device=dev)
+            for label, e in (("clamped gate", ops.ClampedGate(7.0)), ("silu gate", "swiglu")):
+                add(f"linear, {label} ({tag})", n, timed(lambda: ops.linear(x, w_sh, act, epilogue=e)), (2 * eff * H + n * (H + eff)) * 2, 4 * n * H * eff,
+                    like=None if e != "swiglu" else "linear, clamped gate")
+            del cache, kv, kv_like
+        return rows
+
     sampler = ClockSampler()
     sampler.start()
     sampler.mark()
     sizes = {}
     design_sizes, what = DESIGNS[args.design]
     table = {"senupel": senupel_kernel_table, "zotolix": zotolix_kernel_table, "megerax": megerax_kernel_table,
-             "mererax": mererax_kernel_table}.get(args.design, kernel_table)
+             "mererax": mererax_kernel_table, "letanex": letanex_kernel_table}.get(args.design, kernel_table)
     for name in (args.sizes.split(",") if args.sizes else list(design_sizes)):
         design_cfg, llama_cfg, *closest = design_sizes[name]
         sizes[name] = {args.design: model_numbers(design_cfg), "llama": model_numbers(llama_cfg),

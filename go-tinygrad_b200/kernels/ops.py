@@ -106,6 +106,9 @@ _SIGNATURES = {
     "gtg_attention_diff_bf16": ("attention_diff", [_P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
                                                    _F, _F, _F, _I, _P, _P]),
     "gtg_lightning_scan": ("lightning", [_I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
+    "gtg_lightning_chunks": ("lightning", [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
+    "gtg_lightning_chunks_supports": ("lightning", [_I, _I]),
+    "gtg_lightning_chunk_values": ("lightning", [_I, _I, _I, _I, _I]),
     "gtg_hyper_norm": ("hyper", [_I, _I, _P, _P, _P, _P, _P, _P, _P, _F, _P, _P, _I, _I, _I, _P]),
     "gtg_qkv_finish": ("attention_prep", [_I, _P, _I, _P, _P, _I, _I, _F, _P, _P, _F, _P, _I, _P, _P, _P, _L, _P, _I, _P, _P, _P,
                                           _I, _I, _I, _I, _I, _I, _P]),
@@ -131,6 +134,7 @@ _SIGNATURES = {
 _RESTYPES = {"gtg_attention_decode_scratch_floats": c_longlong,
              "gtg_attention_masked_scratch_floats": c_longlong,
              "gtg_attention_diff_scratch_floats": c_longlong,
+             "gtg_lightning_chunk_values": c_longlong,
              "gtg_gemm_bf16_swapab_scratch_floats": c_longlong}
 
 _FUNCS = {}
@@ -907,6 +911,7 @@ def mlstm_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.T
 
 
 LIGHTNING_MAX_KEY_DIM = 512   # most key channels a head of linear attention may have (16 rows a lane, 32 lanes)
+LIGHTNING_CHUNK_TOKENS = 8    # steps that bring at least so many tokens a sequence take the tensor-core kernels
 
 
 def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
@@ -914,7 +919,8 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     """Linear attention with a fixed decay per head (csrc/lightning.cu): S <- decay S + k v^T, out = S^T q;
     q, k [n, heads * d] and v [n, heads * dv], columns of one matrix; decay float32 [heads]; state float32
     [slots, heads, d, dv], read and left per sequence; out float32 [n, heads * dv].  `ctx`: the step's
-    context (rows, sequences, slots)."""
+    context (rows, sequences, slots).  bfloat16 prompts whose heads are a multiple of 8 channels, up to
+    256 of a key, run chunk by chunk on the tensor cores; other steps token by token."""
     for name, t in (("q", q), ("k", k), ("v", v), ("out", out)):
         _rows2d(t, f"lightning_scan: {name}")
     heads = decay.numel()
@@ -928,6 +934,13 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     _need(d <= LIGHTNING_MAX_KEY_DIM, f"lightning_scan: heads of {d} key channels exceed {LIGHTNING_MAX_KEY_DIM}")
     _int32("lightning_scan", ctx.cu_seqlens, ctx.slots)
     _need(n == ctx.n_tokens, "lightning_scan: as many rows as the step has tokens")
+    if (q.dtype == torch.bfloat16 and ctx.max_q_len >= LIGHTNING_CHUNK_TOKENS and _fn("gtg_lightning_chunks_supports")(d, dv)
+            and q.stride(0) % 8 == 0 and out.stride(0) % 2 == 0 and out.data_ptr() % 8 == 0 and all(t.data_ptr() % 16 == 0 for t in (q, k, v))):
+        chunks = ctx.rt.empty(int(_fn("gtg_lightning_chunk_values")(n, ctx.n_seqs, heads, d, dv)), dtype=torch.bfloat16)
+        _check(_fn("gtg_lightning_chunks")(_ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), _ptr(state), _ptr(chunks), _ptr(out), out.stride(0),
+                                           _ptr(ctx.cu_seqlens), _ptr(ctx.slots), int(ctx.n_seqs), int(ctx.max_q_len), heads, d, dv, _stream()),
+               "lightning_scan(chunks)")
+        return
     _check(_fn("gtg_lightning_scan")(_dt(q), _ptr(q), _ptr(k), _ptr(v), q.stride(0), _ptr(decay), _ptr(state), _ptr(out), out.stride(0),
                                      _ptr(ctx.cu_seqlens), _ptr(ctx.slots), int(ctx.n_seqs), heads, d, dv, 1 if ctx.is_decode else 0,
                                      _stream()), "lightning_scan")
