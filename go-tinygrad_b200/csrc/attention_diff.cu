@@ -395,6 +395,224 @@ attention_diff_mma_kernel(const bf16* __restrict__ q, int ldq, bf16* __restrict_
     }
 }
 
+// ---------------------------------------------------------------- decode steps
+// A step in which every sequence brings one token: the (head of the group) rows of a block are at most sixteen, one
+// fragment, so the eight warps share the page instead: warp (map, quarter) scores its map's rows against the page's keys
+// 16 quarter .. + 16 and keeps a running maximum, sum and output of its own; nothing meets across warps until the last
+// page.  One block per (share of the pages, key/value head, sequence); pages arrive kRing - 1 ahead.  At the end the four
+// quarters of a map are added up in order, scaled to their common maximum.
+constexpr int kRing = 3;
+
+template <int DKP, int DVP>
+constexpr int diff_decode_smem_bytes() {
+    constexpr int ring = kRing * kTileRows * (2 * DKP + DVP) * 2, parts = 8 * 16 * (DVP + 4) * 4 + 8 * 16 * 8;
+    return 2 * 16 * DKP * 2 + (ring > parts ? ring : parts);
+}
+
+template <int DKP, int DVP>
+__global__ void __launch_bounds__(kThreads, DVP > 128 ? 1 : 2)
+attention_diff_decode_kernel(const bf16* __restrict__ q, int ldq, bf16* __restrict__ out, int ldo,
+                             const bf16* __restrict__ kc, const bf16* __restrict__ vc, long long page_stride,
+                             const int* __restrict__ block_table, int table_stride,
+                             const int* __restrict__ slots, const int* __restrict__ start_pos,
+                             int n_heads, int n_kv, int d, int vd, float scale, int window,
+                             float lambda, float out_scale, float eps, int n_splits,
+                             float* __restrict__ part_o, float* __restrict__ part_ml) {
+    chain_release();
+    chain_wait();
+    constexpr int KCPR = DKP / 8, VCPR = DVP / 8;
+    constexpr int KTILE = kTileRows * DKP * 2, STAGE = 2 * KTILE + kTileRows * DVP * 2, QTILE = 16 * DKP * 2;
+    constexpr int OPITCH = DVP + 4;
+    extern __shared__ __align__(128) unsigned char smem[];
+    const uint32_t sQ = smem_u32(smem);                    // [map]
+    const uint32_t sR = sQ + 2 * QTILE;                    // [stage]: keys of both maps, values
+    const int b = blockIdx.z, kvh = blockIdx.y, split = blockIdx.x;
+    const int group = n_heads / n_kv, pos = start_pos[b];
+    const int* table = block_table + (size_t)slots[b] * table_stride;
+    const int tid = threadIdx.x, warp = tid >> 5, map = warp >> 2, quarter = warp & 3, lane = tid & 31;
+    const int g = lane >> 2, t4 = lane & 3;
+    const int lo = first_seen(pos, window);
+    const int p_first = lo / kPageTokens, p_last = pos / kPageTokens;
+    const int per_split = (p_last - p_first + n_splits) / n_splits;
+    const int j_lo = p_first + split * per_split;
+    const int j_hi = min(p_last, j_lo + per_split - 1);
+    const size_t th0 = (size_t)b * n_heads + kvh * group;  // (token, head) of row 0
+    if (j_lo > j_hi) {
+        if (tid < 2 * group) {
+            const size_t pidx = ((th0 + tid % group) * 2 + tid / group) * n_splits + split;
+            part_ml[pidx * 2] = -INFINITY;
+            part_ml[pidx * 2 + 1] = 0.f;
+        }
+        return;
+    }
+    for (int id = tid; id < 2 * 16 * KCPR; id += kThreads) {
+        const int mp = id / (16 * KCPR), r = id / KCPR % 16, c = id % KCPR;
+        const bool ok = r < group && c * 8 < d;
+        cp_async16(sQ + mp * QTILE + swz_offset<DKP>(r, c), ok ? q + (size_t)b * ldq + (size_t)(kvh * group + r) * 2 * d + mp * d + c * 8 : q, ok ? 16 : 0);
+    }
+    auto load_page = [&](int stage, int j) {
+        const size_t page = (size_t)table[j] * page_stride;
+        const size_t kbase = page + (size_t)kvh * kPageTokens * 2 * d, vbase = page + (size_t)kvh * kPageTokens * vd;
+        const uint32_t sK = sR + stage * STAGE, sV = sK + 2 * KTILE;
+        for (int id = tid; id < 2 * kTileRows * KCPR; id += kThreads) {
+            const int r = id / (2 * KCPR), mp = id / KCPR % 2, c = id % KCPR;
+            const bool ok = j * kPageTokens + r <= pos && c * 8 < d;
+            cp_async16(sK + mp * KTILE + swz_offset<DKP>(r, c), kc + (ok ? kbase + (size_t)r * 2 * d + mp * d + c * 8 : 0), ok ? 16 : 0);
+        }
+        for (int id = tid; id < kTileRows * VCPR; id += kThreads) {
+            const int r = id / VCPR, c = id % VCPR;
+            const bool ok = j * kPageTokens + r <= pos && c * 8 < vd;
+            cp_async16(sV + swz_offset<DVP>(r, c), vc + (ok ? vbase + (size_t)r * vd + c * 8 : 0), ok ? 16 : 0);
+        }
+    };
+#pragma unroll
+    for (int s = 0; s < kRing - 1; ++s) {                  // the first group holds the queries too; empty groups keep the count
+        if (j_lo + s <= j_hi) load_page(s, j_lo + s);
+        cp_async_commit();
+    }
+    uint32_t qf[DKP / 16][4];
+    float o[DVP / 8][4];
+#pragma unroll
+    for (int i = 0; i < DVP / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+    float m_row[2] = {-INFINITY, -INFINITY}, l_row[2] = {0.f, 0.f};
+    const float s_in = scale * kLog2e;
+    for (int j = j_lo, it = 0; j <= j_hi; ++j, ++it) {
+        cp_async_wait<kRing - 2>();
+        __syncthreads();                                   // this page stands; the page before it has been read
+        if (j + kRing - 1 <= j_hi) load_page((it + kRing - 1) % kRing, j + kRing - 1);
+        cp_async_commit();
+        if (it == 0) {
+#pragma unroll
+            for (int kk = 0; kk < DKP / 16; ++kk) {
+                const int r = (lane & 7) + ((lane >> 3) & 1) * 8, c = kk * 2 + (lane >> 4);
+                ldmatrix_x4(qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3], sQ + map * QTILE + swz_offset<DKP>(r, c));
+            }
+        }
+        const int key0 = j * kPageTokens + quarter * 16;
+        if (key0 > pos || key0 + 15 < lo) continue;        // none of the warp's sixteen keys is seen
+        const uint32_t kbase = sR + (it % kRing) * STAGE + map * KTILE, vbase = sR + (it % kRing) * STAGE + 2 * KTILE;
+        float s[2][4];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) { s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f; }
+#pragma unroll
+        for (int kk = 0; kk < DKP / 16; ++kk) {
+            uint32_t b0, b1, b2, b3;
+            const int r = quarter * 16 + (lane & 7) + (lane >> 4) * 8, c = kk * 2 + ((lane >> 3) & 1);
+            ldmatrix_x4(b0, b1, b2, b3, kbase + swz_offset<DKP>(r, c));
+            mma_bf16_16816(s[0], qf[kk], b0, b1);
+            mma_bf16_16816(s[1], qf[kk], b2, b3);
+        }
+        if (key0 + 15 > pos || key0 < lo) {
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int key = key0 + i * 8 + t4 * 2 + (e & 1);
+                    if (key > pos || key < lo) s[i][e] = -INFINITY;
+                }
+        }
+        float corr[2];
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            float mx = fmaxf(fmaxf(s[0][r * 2], s[0][r * 2 + 1]), fmaxf(s[1][r * 2], s[1][r * 2 + 1]));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+            const float m_new = fmaxf(m_row[r], mx * s_in);        // finite: at least one of the keys is seen
+            corr[r] = fast_exp2(m_row[r] - m_new);
+            m_row[r] = m_new;
+            float sum = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float p = fast_exp2(fmaf(s[i][r * 2 + e], s_in, -m_new));
+                    s[i][r * 2 + e] = p;
+                    sum += p;
+                }
+            l_row[r] = l_row[r] * corr[r] + sum;
+        }
+        const uint32_t pa[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
+#pragma unroll
+        for (int dd = 0; dd < DVP / 16; ++dd) {
+            uint32_t b0, b1, b2, b3;
+            const int r = quarter * 16 + ((lane >> 3) & 1) * 8 + (lane & 7), c = dd * 2 + (lane >> 4);
+            ldmatrix_x4_trans(b0, b1, b2, b3, vbase + swz_offset<DVP>(r, c));
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                float* oo = o[dd * 2 + x];
+                oo[0] *= corr[0]; oo[1] *= corr[0]; oo[2] *= corr[1]; oo[3] *= corr[1];
+            }
+            mma_bf16_16816(o[dd * 2], pa, b0, b1);
+            mma_bf16_16816(o[dd * 2 + 1], pa, b2, b3);
+        }
+    }
+    cp_async_wait<0>();
+    __syncthreads();                                       // the ring has been read: its place takes the warps' parts
+    float* po = reinterpret_cast<float*>(smem + 2 * QTILE);                // [warp][16][OPITCH]
+    float2* pml = reinterpret_cast<float2*>(po + 8 * 16 * OPITCH);         // [warp][16]
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        l_row[r] += __shfl_xor_sync(0xffffffffu, l_row[r], 1);
+        l_row[r] += __shfl_xor_sync(0xffffffffu, l_row[r], 2);
+        const int row = g + r * 8;
+        if (row >= group) continue;
+        float* dst = po + (warp * 16 + row) * OPITCH + t4 * 2;
+#pragma unroll
+        for (int i = 0; i < DVP / 8; ++i) *reinterpret_cast<float2*>(dst + i * 8) = make_float2(o[i][r * 2], o[i][r * 2 + 1]);
+        if (t4 == 0) pml[warp * 16 + row] = make_float2(m_row[r], l_row[r]);
+    }
+    __syncthreads();
+    // a warp a row: the quarters of both maps, then the share or the finished head
+    for (int row = warp; row < group; row += 8) {
+        float f[2][4], M[2], L[2];
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+            M[mp] = -INFINITY;
+            L[mp] = 0.f;
+#pragma unroll
+            for (int k = 0; k < 4; ++k) M[mp] = fmaxf(M[mp], pml[(mp * 4 + k) * 16 + row].x);
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                const float2 ml = pml[(mp * 4 + k) * 16 + row];
+                f[mp][k] = ml.x == -INFINITY ? 0.f : exp2f(ml.x - M[mp]);
+                L[mp] += f[mp][k] * ml.y;
+            }
+        }
+        const size_t th = th0 + row;
+        constexpr int PER = DVP / 32;
+        float a[2][PER];
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp)
+#pragma unroll
+            for (int i = 0; i < PER; ++i) {
+                a[mp][i] = 0.f;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) a[mp][i] = fmaf(f[mp][k], po[((mp * 4 + k) * 16 + row) * OPITCH + lane + 32 * i], a[mp][i]);
+            }
+        if (n_splits > 1) {
+#pragma unroll
+            for (int mp = 0; mp < 2; ++mp) {
+                const size_t pidx = (th * 2 + mp) * n_splits + split;
+#pragma unroll
+                for (int i = 0; i < PER; ++i) part_o[pidx * DVP + lane + 32 * i] = a[mp][i];
+                if (lane == 0) { part_ml[pidx * 2] = M[mp]; part_ml[pidx * 2 + 1] = L[mp]; }
+            }
+            continue;
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            a[0][i] = a[0][i] / L[0] - lambda * (a[1][i] / L[1]);
+            ss = fmaf(a[0][i], a[0][i], ss);
+        }
+        const float inv = out_scale / sqrtf(warp_sum(ss) / (float)vd + eps);
+        bf16* dst = out + (size_t)b * ldo + (size_t)(kvh * group + row) * vd;
+#pragma unroll
+        for (int i = 0; i < PER; ++i)
+            if (lane + 32 * i < vd) dst[lane + 32 * i] = __float2bfloat16_rn(a[0][i] * inv);
+    }
+}
+
 // One block per (token, query head), a thread per channel: each map's shares in order, scaled to their
 // common maximum; then the difference and its norm.
 __global__ void attention_diff_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
@@ -431,12 +649,28 @@ inline int padded(int d) { return d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 
 struct DiffArgs {
     const bf16* q; int ldq; bf16* out; int ldo; const bf16 *kc, *vc; long long page_stride; const int* block_table; int table_stride;
-    const int *cu_seqlens, *slots, *start_pos; int n_seqs, tiles, n_heads, n_kv, d, vd; float scale; int window;
+    const int *cu_seqlens, *slots, *start_pos; int n_seqs, max_q_len, tiles, n_heads, n_kv, d, vd; float scale; int window;
     float lambda, out_scale, eps; int n_splits; float *part_o, *part_ml; cudaStream_t stream;
 };
 
 template <int DKP, int DVP>
+int launch_diff_decode(const DiffArgs& a) {
+    auto kernel = attention_diff_decode_kernel<DKP, DVP>;
+    constexpr int smem = diff_decode_smem_bytes<DKP, DVP>();
+    static bool configured = false;
+    if (!configured) {
+        const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        if (e != cudaSuccess) return (int)e;
+        configured = true;
+    }
+    return launch_chained(kernel, dim3(a.n_splits, a.n_kv, a.n_seqs), dim3(kThreads), smem, a.stream, a.q, a.ldq, a.out, a.ldo,
+                          a.kc, a.vc, a.page_stride, a.block_table, a.table_stride, a.slots, a.start_pos, a.n_heads, a.n_kv,
+                          a.d, a.vd, a.scale, a.window, a.lambda, a.out_scale, a.eps, a.n_splits, a.part_o, a.part_ml);
+}
+
+template <int DKP, int DVP>
 int launch_diff(const DiffArgs& a) {
+    if (a.max_q_len == 1 && a.n_heads / a.n_kv <= 16) return launch_diff_decode<DKP, DVP>(a);
     auto kernel = attention_diff_mma_kernel<DKP, DVP>;
     constexpr int smem = diff_smem_bytes<DKP, DVP>();
     static bool configured = false;
@@ -515,7 +749,7 @@ GTG_API int gtg_attention_diff_bf16(const void* q, int ldq, void* out, int ldo, 
     if (tiles * n_splits > 0x7fffffffLL || n_seqs > 65535 || n_kv > 65535) return kErrUnsupported;
     const int dvp = padded(vd);
     const DiffArgs a{(const bf16*)q, ldq, (bf16*)out, ldo, (const bf16*)kc, (const bf16*)vc, page_stride, block_table, table_stride,
-                     cu_seqlens, slots, start_pos, n_seqs, (int)tiles, n_heads, n_kv, d, vd, scale, window, lambda, out_scale, eps,
+                     cu_seqlens, slots, start_pos, n_seqs, max_q_len, (int)tiles, n_heads, n_kv, d, vd, scale, window, lambda, out_scale, eps,
                      n_splits, scratch, scratch ? scratch + (size_t)n_tokens * n_heads * 2 * n_splits * dvp : nullptr, stream};
     int st;
     if (d <= 64) st = dvp == 64 ? launch_diff<64, 64>(a) : dvp == 128 ? launch_diff<64, 128>(a) : launch_diff<64, 256>(a);

@@ -610,11 +610,25 @@ GTG_API int gtg_add_layernorm(int dtype, float* residual, const void* pending, c
 // sublayer stands between two norms, the second of which meets the first of the next sublayer here.
 // U is the update's type (float from a product that kept its sums).  Rows as in add_rmsnorm: with `rows`
 // nothing is written back.  Everything in float.
+//
+// With `ex.top` > 0 the update is that of a mixture of experts and is summed here: of row r, the weighted sum of its
+// experts' rows ex.y[ex.item_row[r top + k],:] (an item without a row: of the mixture's input ex.x[r,:]), k in order, and
+// ex.base[r,:] last; `update` is then not read.
+struct ExpertRows {
+    const float* y;
+    int ldy;
+    const int* item_row;
+    const float* weights;
+    const void* x;               // of the output's type, or null
+    int ldx;
+    const float* base;           // or null
+    int top;
+};
 template <typename U, typename T>
 __global__ void layernorm_add_layernorm_kernel(float* __restrict__ residual, const U* __restrict__ update,
                                                const float* __restrict__ weight_u, float eps_u,
                                                const float* __restrict__ weight, const float* __restrict__ bias, float eps,
-                                               T* __restrict__ out, const int* __restrict__ rows, int H) {
+                                               T* __restrict__ out, const int* __restrict__ rows, int H, ExpertRows ex) {
     chain_release();
     chain_wait();
     extern __shared__ float smem[];
@@ -635,7 +649,17 @@ __global__ void layernorm_add_layernorm_kernel(float* __restrict__ residual, con
     };
     float sum = 0.f, mean;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        const float u = to_f32<U>(up[i]);
+        float u = 0.f;
+        if (ex.top > 0) {
+            for (int k = 0; k < ex.top; ++k) {
+                const int er = ex.item_row[(size_t)r * ex.top + k];
+                const float v = er >= 0 ? ex.y[(size_t)er * ex.ldy + i] : to_f32<T>(reinterpret_cast<const T*>(ex.x)[(size_t)r * ex.ldx + i]);
+                u = fmaf(ex.weights[(size_t)r * ex.top + k], v, u);
+            }
+            if (ex.base) u += ex.base[(size_t)r * H + i];
+        } else {
+            u = to_f32<U>(up[i]);
+        }
         row[i] = u;
         sum += u;
     }
@@ -682,12 +706,12 @@ __device__ __forceinline__ void load_eight(const bf16* p, float* x) {
 
 // The same for bfloat16 rows whose width is a multiple of 8 and at most 8192: every thread owns 8
 // consecutive channels, kept in registers from the first read to the last write.
-template <typename U>
+template <typename U, bool kExperts>
 __global__ void __launch_bounds__(1024)
 layernorm_add_layernorm_vec_kernel(float* __restrict__ residual, const U* __restrict__ update,
                                    const float* __restrict__ weight_u, float eps_u,
                                    const float* __restrict__ weight, const float* __restrict__ bias, float eps,
-                                   bf16* __restrict__ out, const int* __restrict__ rows, int H) {
+                                   bf16* __restrict__ out, const int* __restrict__ rows, int H, ExpertRows ex) {
     chain_release();
     chain_wait();        // before every load: one through a restricted pointer to const may be moved over a later wait
     __shared__ float part[4][32];
@@ -705,8 +729,29 @@ layernorm_add_layernorm_vec_kernel(float* __restrict__ residual, const U* __rest
     float* rp = residual + (size_t)r * H + c;
     float sum = 0.f;
     if (active) {
-        load_eight(update + (size_t)r * H + c, u);
         load_eight(rp, x);
+        if constexpr (kExperts) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) u[j] = 0.f;
+#pragma unroll 4
+            for (int k = 0; k < ex.top; ++k) {
+                const int er = ex.item_row[(size_t)r * ex.top + k];
+                const float f = ex.weights[(size_t)r * ex.top + k];
+                float v[8];
+                if (er >= 0) load_eight(ex.y + (size_t)er * ex.ldy + c, v);
+                else load_eight(reinterpret_cast<const bf16*>(ex.x) + (size_t)r * ex.ldx + c, v);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) u[j] = fmaf(f, v[j], u[j]);
+            }
+            if (ex.base) {
+                float v[8];
+                load_eight(ex.base + (size_t)r * H + c, v);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) u[j] += v[j];
+            }
+        } else {
+            load_eight(update + (size_t)r * H + c, u);
+        }
 #pragma unroll
         for (int j = 0; j < 8; ++j) sum += u[j];
     }
@@ -745,17 +790,24 @@ layernorm_add_layernorm_vec_kernel(float* __restrict__ residual, const U* __rest
 
 GTG_API int gtg_layernorm_add_layernorm(int dtype, int update_f32, float* residual, const void* update, const float* weight_u,
                                         float eps_u, const float* weight, const float* bias, float eps, void* out,
-                                        const int* rows, int R, int H, cudaStream_t stream) {
+                                        const int* rows, int R, int H, const float* y, int ldy, const int* item_row,
+                                        const float* expert_weights, const void* x, int ldx, const float* base, int top,
+                                        cudaStream_t stream) {
     if (R <= 0) return 0;
-    if (H <= 0 || !update || !weight_u || !weight) return kErrBadArgument;
-    if (dtype == 1 && H % 8 == 0 && H <= 8192 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
+    if (H <= 0 || (!update && top <= 0) || !weight_u || !weight) return kErrBadArgument;
+    if (top > 0 && (!y || ldy < H || !item_row || !expert_weights || (x && ldx < H))) return kErrBadArgument;
+    const ExpertRows ex{y, ldy, item_row, expert_weights, x, ldx, base, top};
+    const bool ex_wide = top <= 0 || (ldy % 4 == 0 && ldx % 8 == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)x % 16) == 0 && ((uintptr_t)base % 16) == 0);
+    if (ex_wide && dtype == 1 && H % 8 == 0 && H <= 8192 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
         ((uintptr_t)weight % 16) == 0 && ((uintptr_t)weight_u % 16) == 0 && ((uintptr_t)bias % 16) == 0 && ((uintptr_t)update % 16) == 0) {
         const int t = ((H / 8) + 31) / 32 * 32;
-        if (update_f32)
-            return launch_chained(layernorm_add_layernorm_vec_kernel<float>, dim3(R), dim3(t), 0, stream, residual, (const float*)update,
-                                  weight_u, eps_u, weight, bias, eps, (bf16*)out, rows, H);
-        return launch_chained(layernorm_add_layernorm_vec_kernel<bf16>, dim3(R), dim3(t), 0, stream, residual, (const bf16*)update,
-                              weight_u, eps_u, weight, bias, eps, (bf16*)out, rows, H);
+#define GTG_NORM_ADD_NORM_VEC(U, EX)                                                                             \
+        return launch_chained(layernorm_add_layernorm_vec_kernel<U, EX>, dim3(R), dim3(t), 0, stream, residual, (const U*)update, \
+                              weight_u, eps_u, weight, bias, eps, (bf16*)out, rows, H, ex)
+        if (top > 0) GTG_NORM_ADD_NORM_VEC(float, true);
+        if (update_f32) GTG_NORM_ADD_NORM_VEC(float, false);
+        GTG_NORM_ADD_NORM_VEC(bf16, false);
+#undef GTG_NORM_ADD_NORM_VEC
     }
     int threads = 32;
     while (threads < 1024 && threads * 4 < H) threads *= 2;
@@ -768,7 +820,7 @@ GTG_API int gtg_layernorm_add_layernorm(int dtype, int update_f32, float* residu
             if (e != cudaSuccess) return (int)e;                                                                 \
         }                                                                                                        \
         return launch_chained(layernorm_add_layernorm_kernel<U, T>, dim3(R), dim3(threads), smem, stream, residual, (const U*)update, \
-                              weight_u, eps_u, weight, bias, eps, (T*)out, rows, H);                             \
+                              weight_u, eps_u, weight, bias, eps, (T*)out, rows, H, ex);                         \
     } while (0)
     if (dtype == 0) GTG_NORM_ADD_NORM(float, float);
     if (dtype == 1 && update_f32) GTG_NORM_ADD_NORM(float, bf16);

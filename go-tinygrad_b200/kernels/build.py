@@ -32,6 +32,7 @@ LIBRARIES: Dict[str, str] = {
     "gemm_f32": "gemm_f32.cu",
     "attention_simple": "attention_simple.cu",
     "attention_diff": "attention_diff.cu",
+    "attention_diff_tcgen05": "attention_diff_tcgen05.cu",
     "lightning": "lightning.cu",
     "sampling": "sampling.cu",
     "gemm_bf16_mma": "gemm_bf16_mma.cu",

@@ -32,7 +32,7 @@ _SIGNATURES = {
     "gtg_rope_table": ("elementwise", [_P, _P, _P, _I, _I, _D, _P]),
     "gtg_rope_kv_store": ("elementwise", [_I, _P, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _P]),
     "gtg_add_layernorm": ("elementwise", [_I, _P, _P, _P, _P, _F, _P, _P, _I, _I, _P]),
-    "gtg_layernorm_add_layernorm": ("elementwise", [_I, _I, _P, _P, _P, _F, _P, _P, _F, _P, _P, _I, _I, _P]),
+    "gtg_layernorm_add_layernorm": ("elementwise", [_I, _I, _P, _P, _P, _F, _P, _P, _F, _P, _P, _I, _I, _P, _I, _P, _P, _P, _I, _P, _I, _P]),
     "gtg_activation": ("elementwise", [_I, _P, _I, _I, _I, _I, _P]),
     "gtg_softcap": ("elementwise", [_P, _L, _F, _P]),
     "gtg_hidden_concat": ("elementwise", [_I, _P, _P, _P, _P, _I, _I, _P]),
@@ -105,6 +105,11 @@ _SIGNATURES = {
     "gtg_attention_diff_splits": ("attention_diff", [_I, _I, _I, _I, _I, _I]),
     "gtg_attention_diff_bf16": ("attention_diff", [_P, _I, _P, _I, _P, _P, _L, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I,
                                                    _F, _F, _F, _I, _P, _P]),
+    "gtg_attention_diff_tcgen05_supports": ("attention_diff_tcgen05", [_I, _I]),
+    "gtg_attention_diff_tcgen05_status": ("attention_diff_tcgen05", []),
+    "gtg_attention_diff_tcgen05_test_hooks": ("attention_diff_tcgen05", [_I]),
+    "gtg_attention_diff_tcgen05": ("attention_diff_tcgen05", [_P, _I, _I, _P, _I, _P, _P, _L, _I, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I,
+                                                              _F, _I, _F, _F, _F, _P]),
     "gtg_lightning_scan": ("lightning", [_I, _P, _P, _P, _I, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
     "gtg_lightning_chunks": ("lightning", [_P, _P, _P, _I, _P, _P, _P, _P, _I, _P, _P, _I, _I, _I, _I, _I, _P]),
     "gtg_lightning_chunks_supports": ("lightning", [_I, _I]),
@@ -452,26 +457,57 @@ def add_layernorm(residual: torch.Tensor, pending: Optional[torch.Tensor], weigh
                                     _ptr(out), _ptr(rows), R, H, _stream()), "add_layernorm")
 
 
-def layernorm_add_layernorm(residual: torch.Tensor, update: torch.Tensor, update_weight: torch.Tensor, update_eps: float,
+@dataclass
+class ExpertSum:
+    """A mixture's update that has not been summed yet: what `moe_combine` takes.  A norm kernel that reads it adds
+    the rows up itself."""
+    y: torch.Tensor
+    item_row: torch.Tensor
+    weights: torch.Tensor
+    x: Optional[torch.Tensor]
+    base: Optional[torch.Tensor]
+
+    def float(self) -> torch.Tensor:
+        """The update as a float32 tensor."""
+        out = torch.empty(self.weights.shape[0], self.y.shape[1], dtype=torch.float32, device=self.y.device)
+        moe_combine(self.y, self.item_row, self.weights, out, x=self.x, base=self.base)
+        return out
+
+
+def layernorm_add_layernorm(residual: torch.Tensor, update, update_weight: torch.Tensor, update_eps: float,
                             weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out: torch.Tensor,
                             rows: Optional[torch.Tensor] = None) -> None:
     """residual += LN(update) * update_weight; out = LN(residual) * weight (+ bias), LN(x) = (x - mean) /
-    sqrt(var + eps), all in float.  `update` is float32 or of out's dtype.  With `rows` only those rows are
+    sqrt(var + eps), all in float.  `update` is float32 or of out's dtype, or an `ExpertSum`.  With `rows` only those rows are
     read (nothing is written back) and out has len(rows) rows."""
     H = residual.shape[1]
     R = rows.numel() if rows is not None else residual.shape[0]
     _need(residual.dtype == torch.float32 and residual.is_contiguous(), "layernorm_add_layernorm: residual must be contiguous float32")
-    _need(update.is_contiguous() and update.shape == residual.shape and update.dtype in (torch.float32, out.dtype),
-          "layernorm_add_layernorm: update must be contiguous [N, H], float32 or of out's dtype")
+    experts = (None, 0, None, None, None, 0, None, 0)
+    update_f32 = True
+    if isinstance(update, ExpertSum):
+        e, N = update, residual.shape[0]
+        top = e.weights.shape[1]
+        _need(e.y.dtype == torch.float32 and e.y.shape[1] == H and e.y.stride(1) == 1 and e.item_row.dtype == torch.int32 and e.item_row.is_contiguous()
+              and e.item_row.numel() == N * top and e.weights.dtype == torch.float32 and e.weights.is_contiguous() and e.weights.shape[0] == N
+              and (e.x is None or (e.x.dtype == out.dtype and tuple(e.x.shape) == (N, H) and e.x.stride(1) == 1))
+              and (e.base is None or (e.base.dtype == torch.float32 and e.base.is_contiguous() and tuple(e.base.shape) == (N, H))),
+              "layernorm_add_layernorm: the experts' rows do not fit the hidden state")
+        experts = (_ptr(e.y), e.y.stride(0), _ptr(e.item_row), _ptr(e.weights), _ptr(e.x), e.x.stride(0) if e.x is not None else 0, _ptr(e.base), top)
+        update = None
+    else:
+        _need(update.is_contiguous() and update.shape == residual.shape and update.dtype in (torch.float32, out.dtype),
+              "layernorm_add_layernorm: update must be contiguous [N, H], float32 or of out's dtype")
+        update_f32 = update.dtype == torch.float32
     for name, t in (("update_weight", update_weight), ("weight", weight), ("bias", bias)):
         _need((t is None and name == "bias") or (t is not None and t.dtype == torch.float32 and t.is_contiguous() and t.numel() == H),
               f"layernorm_add_layernorm: {name} must be float32 [H]")
     _need(out.is_contiguous() and tuple(out.shape) == (R, H), "layernorm_add_layernorm: out must be contiguous [rows, H]")
     if rows is not None:
         _need(rows.dtype == torch.int32 and rows.is_contiguous(), "layernorm_add_layernorm: rows must be contiguous int32")
-    _check(_fn("gtg_layernorm_add_layernorm")(_dt(out), 1 if update.dtype == torch.float32 else 0, _ptr(residual), _ptr(update),
+    _check(_fn("gtg_layernorm_add_layernorm")(_dt(out), 1 if update_f32 else 0, _ptr(residual), _ptr(update),
                                               _ptr(update_weight), float(update_eps), _ptr(weight), _ptr(bias), float(eps), _ptr(out),
-                                              _ptr(rows), R, H, _stream()), "layernorm_add_layernorm")
+                                              _ptr(rows), R, H, *experts, _stream()), "layernorm_add_layernorm")
 
 
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2}
@@ -1248,13 +1284,13 @@ def bounded_wait_failures() -> int:
     copies (it then returned without a result).  Reading it synchronises."""
     total = 0
     for symbol in ("gtg_gemm_bf16_skinny_status", "gtg_gemm_bf16_tcgen05_status", "gtg_gemm_bf16_swapab_status",
-                   "gtg_attention_tcgen05_status", "gtg_latent_status"):
+                   "gtg_attention_tcgen05_status", "gtg_attention_diff_tcgen05_status", "gtg_latent_status"):
         if _SIGNATURES[symbol][0] in build._LOADED:        # only libraries that have run can have failed
             total += int(_fn(symbol)())
     return total
 
 
-WAITING_LIBRARIES = ("gemm_bf16_skinny", "gemm_bf16_tcgen05", "gemm_bf16_swapab", "attention_tcgen05", "latent")
+WAITING_LIBRARIES = ("gemm_bf16_skinny", "gemm_bf16_tcgen05", "gemm_bf16_swapab", "attention_tcgen05", "attention_diff_tcgen05", "latent")
 
 
 def wait_test_hooks(library: str, test_waits: bool) -> None:
@@ -1452,9 +1488,39 @@ def attention_diff_bf16(q: torch.Tensor, out: torch.Tensor, kv, cu_seqlens, slot
            "attention_diff_bf16")
 
 
+def attention_diff_tcgen05_supports(kv) -> bool:
+    """Whether `attention_diff_tcgen05` takes this cache entry: maps of 64 channels over values of 128,
+    keys and values lying page by page as [k|v][head][token][channel]."""
+    return (kv.k.dtype == torch.bfloat16 and kv.head_dim == kv.value_dim == 128
+            and bool(_fn("gtg_attention_diff_tcgen05_supports")(kv.head_dim // 2, kv.value_dim))
+            and kv.page_stride == 2 * kv.n_kv_heads * 64 * 128 and kv.v.data_ptr() - kv.k.data_ptr() == kv.n_kv_heads * 64 * 128 * 2)
+
+
+def attention_diff_tcgen05(q: torch.Tensor, out: torch.Tensor, kv, cu_seqlens, slots, start_pos, n_seqs: int, max_q_len: int,
+                           n_heads: int, scale: float, lam: float, out_scale: float, eps: float, window: int = 0) -> None:
+    """Differential attention of prompts on tcgen05 (128 queries x one head with both its maps per thread block)."""
+    _rows2d(q, "attention: q"); _rows2d(out, "attention: out")
+    _need(q.dtype == torch.bfloat16 and out.dtype == torch.bfloat16 and attention_diff_tcgen05_supports(kv), "attention_diff_tcgen05: cache entry not supported")
+    _need(q.shape[1] >= n_heads * 128 and out.shape[1] >= n_heads * 128, "attention: q or out is too narrow")
+    _int32("attention_diff", cu_seqlens, slots, start_pos)
+    _check_access("attention_diff_tcgen05", 2, kv, slots, start_pos=start_pos, cu_seqlens=cu_seqlens, n_items=n_seqs)
+    _check(_fn("gtg_attention_diff_tcgen05")(_ptr(q), q.stride(0), q.shape[0], _ptr(out), out.stride(0), _ptr(kv.k), _ptr(kv.v), kv.page_stride,
+                                             kv.k.shape[0], _ptr(kv.block_table), kv.table_stride, _ptr(cu_seqlens), _ptr(slots),
+                                             _ptr(start_pos), int(n_seqs), int(max_q_len), n_heads, kv.n_kv_heads, 64, 128, float(scale),
+                                             int(window), float(lam), float(out_scale), float(eps), _stream()), "attention_diff_tcgen05")
+
+
+DIFF_TCGEN05_TOKENS = 64      # steps that bring more tokens a sequence take the tcgen05 kernel where it knows the sizes
+
+
 def attention_diff(q: torch.Tensor, out: torch.Tensor, kv, ctx, n_heads: int, scale: float, lam: float, out_scale: float,
                    eps: float, window: int = 0) -> None:
     """Differential attention of a step (`ctx`: its context) by the kernel that takes its sizes."""
+    if (q.dtype == torch.bfloat16 and ctx.max_q_len > DIFF_TCGEN05_TOKENS and attention_diff_tcgen05_supports(kv) and scale > 0
+            and q.stride(0) % 8 == 0 and out.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
+        attention_diff_tcgen05(q, out, kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, ctx.n_seqs, ctx.max_q_len, n_heads, scale, lam,
+                               out_scale, eps, window)
+        return
     if (q.dtype == torch.bfloat16 and attention_diff_supports(kv) and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0
             and out.stride(0) % 2 == 0 and scale > 0):
         splits = int(_fn("gtg_attention_diff_splits")(ctx.n_seqs, ctx.max_q_len, n_heads, kv.n_kv_heads, ctx.max_kv_len, int(window)))

@@ -204,6 +204,9 @@ class StepContext:
     # set by a block whose norm takes a sublayer's update in float32: a part whose last step
     # leaves float sums may then return them unrounded instead of in the compute dtype
     float_updates: bool = False
+    # set by a block whose next norm can sum a mixture's rows itself: a routed feed-forward may then return
+    # them as an `ops.ExpertSum` instead of their sum
+    expert_sums: bool = False
     # with float_updates: a bias (float32 [H]) that the part leaves for the block's norm kernel to add to
     # the update it returns, instead of adding it itself; the block takes it and sets this None again
     update_bias: Optional[torch.Tensor] = None
@@ -293,7 +296,8 @@ class ResidualStream:
 
     `pending_norm`, where set, is a layer norm (weight, eps) that the pending update passes before
     it is added: a block whose sublayers stand between two norms leaves it to the next norm, which
-    does both in one pass (`ops.layernorm_add_layernorm`).  The pending update may then be float32."""
+    does both in one pass (`ops.layernorm_add_layernorm`).  The pending update may then be float32,
+    or a mixture's rows that have not been summed yet (`ops.ExpertSum`)."""
 
     def __init__(self, residual: torch.Tensor, pending: Optional[torch.Tensor] = None):
         self.residual = residual

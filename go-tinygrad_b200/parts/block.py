@@ -189,11 +189,12 @@ class SandwichNormBlock(Block):
             if self.feed_forward is not None:
                 x = self.feed_forward_norm.forward(stream, ctx)
                 ctx.trace("mlp_input", x)
+                ctx.expert_sums = True
                 stream.pending = self.feed_forward.forward(x, ctx)
                 stream.pending_norm = (self.feed_forward_output_norm.weight, self.feed_forward_output_norm.eps)
-                ctx.trace("down", stream.pending)
+                ctx.trace("down", lambda: stream.pending.float())
         finally:
-            ctx.float_updates = False
+            ctx.float_updates = ctx.expert_sums = False
         ctx.trace("hidden_post_ffn", lambda: _hidden(stream))
 
 

@@ -264,8 +264,11 @@ class RoutedExperts(FeedForward):
             ops.swiglu_bias(sums, None, None, act, epilogue=self.gate)
         y = rt.empty(rows, self.hidden, dtype=torch.float32)
         ops.moe_product(act, row_item, 0, self.w_down, tile_expert, y)
+        base = self._shared_update(x, ctx)
+        if ctx.expert_sums:
+            return ops.ExpertSum(y, item_row, weights, x if self.n_identity else None, base)
         out = rt.empty(n, self.hidden, dtype=torch.float32 if ctx.float_updates else None)
-        ops.moe_combine(y, item_row, weights, out, x=x if self.n_identity else None, base=self._shared_update(x, ctx))
+        ops.moe_combine(y, item_row, weights, out, x=x if self.n_identity else None, base=base)
         return out
 
     def _shared_update(self, x: torch.Tensor, ctx: StepContext) -> Optional[torch.Tensor]:

@@ -113,6 +113,42 @@ def expanded_attention():
     return run, want, dict(rtol=2e-2, atol=2e-2)
 
 
+def differential_attention():
+    """Prompts through both maps of every head: a whole one and a continued one."""
+    from go_tinygrad_b200.cache import Cache, KVRequest
+    heads, n_kv, new, starts = 4, 2, [300, 20], [0, 70]
+    cache = Cache([[KVRequest(n_kv, 128, None, value_dim=128)]], [None], max_tokens=64 * 8, max_slots=3, dtype=BF16, device=torch.device(DEV))
+    slots = [cache.open_sequence() for _ in new]
+    cache.reserve_many([(s, a + n) for s, a, n in zip(slots, starts, new)]); cache.flush_tables()
+    kv = cache.handles[0].kv
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=DEV)
+    q = rnd(sum(new), heads * 128, dtype=BF16, seed=5)
+    want, at = [], 0
+    for b, (s, a, n) in enumerate(zip(slots, starts, new)):
+        k, v = rnd(a + n, n_kv, 128, dtype=BF16, seed=6 + b), rnd(a + n, n_kv, 128, dtype=BF16, seed=8 + b)
+        for p0 in range(0, a + n, 64):
+            page = int(cache.groups[0].table_host[s][p0 // 64])
+            for rows, plane in ((k, kv.k), (v, kv.v)):
+                plane[page, :, : min(64, a + n - p0)] = rows[p0:p0 + 64].transpose(0, 1)
+        for i in range(n):
+            out = []
+            for h in range(heads):
+                qh, kh, vh = q[at + i].double().view(heads, 2, 64)[h], k[: a + i + 1, h // 2].double().view(-1, 2, 64), v[: a + i + 1, h // 2].double()
+                a1, a2 = (torch.softmax(kh[:, m] @ qh[m] * 0.125, dim=0) @ vh for m in range(2))
+                o = a1 - 0.3 * a2
+                out.append(o / torch.sqrt((o * o).mean() + 1e-3) * 0.7)
+            want.append(torch.cat(out))
+        at += n
+    want = torch.stack(want).float()
+
+    def run():
+        out = torch.full((sum(new), heads * 128), 7.0, dtype=BF16, device=DEV)
+        ops.attention_diff_tcgen05(q, out, kv, i32([0, new[0], sum(new)]), i32(slots), i32(starts), 2, max(new), heads, 0.125, 0.3, 0.7, 1e-3)
+        return out.float()
+    run.keep = cache
+    return run, want, dict(rtol=2e-2, atol=2e-2)
+
+
 CASES = {
     # library -> what runs its kernels: (how to build the case)
     "gemm_bf16_tcgen05": [lambda: product("tcgen05", 300, 520, 1024), residual_product],
@@ -123,6 +159,7 @@ CASES = {
                          lambda: product("skinny", 3, 50, 8200),         # an inner size that takes the row-copy kernel,
                          lambda: product("skinny", 5, 96, 264)],         # ... with a cluster of ranks and with one
     "attention_tcgen05": [prompt_attention],
+    "attention_diff_tcgen05": [differential_attention],
     "latent": [latent_attention, expanded_attention],
 }
 

@@ -270,7 +270,64 @@ def test_tensor_core_differential_attention_against_the_plain_kernel(n_heads, n_
         scratch = torch.empty(int(ops._fn("gtg_attention_diff_scratch_floats")(sum(lens), n_heads, vd, splits)) or 1, dtype=torch.float32, device=DEV)
         ops.attention_diff_bf16(q, out, kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, 4, 200, n_heads, scale, lam, out_scale, eps, window, splits, scratch)
         close(out, f64(want), "bfloat16", splits)
+
+
+@pytest.mark.parametrize("n_heads,n_kv,window", [(8, 2, 0), (3, 1, 0), (4, 4, 100), (6, 3, 300)])
+def test_prompt_differential_attention_on_tcgen05_against_the_plain_kernel(n_heads, n_kv, window):
+    """Maps of 64 channels over values of 128: sequences of one token up to several tiles, that start and go on, on slots
+    that are not in order; queries from small to so large that the running maximum jumps again and again."""
+    from go_tinygrad_b200.cache import KVRequest
+    rng = np.random.default_rng(n_heads)
+    rt = Runtime(DEV, torch.bfloat16)
+    starts, lens = [0, 130, 517, 63, 0], [700, 1, 129, 65, 128]
+    caches = {}
+    for dt in (torch.bfloat16, torch.float32):
+        c = Cache([[KVRequest(n_kv, 128, None, value_dim=128)]], [None], max_tokens=64 * 40, max_slots=6, dtype=dt, device=DEV)
+        slots = [c.open_sequence() for _ in range(6)][::-1][:5]
+        c.reserve_many([(s, a + n) for s, a, n in zip(slots, starts, lens)]); c.flush_tables()
+        caches[dt] = c
+    store = caches[torch.bfloat16].groups[0].storage
+    store.copy_(t32(rng.standard_normal(tuple(store.shape))).to(torch.bfloat16))
+    caches[torch.float32].groups[0].storage.copy_(store.float())
+    ctx = context(rt, lens, starts, slots)
+    for size in (0.3, 2.0, 12.0):
+        q = (t32(rng.standard_normal((sum(lens), n_heads * 128))) * size).to(torch.bfloat16)
+        want = torch.empty(sum(lens), n_heads * 128, dtype=torch.float32, device=DEV)
+        args = (n_heads, 0.125, -0.4, 0.7, 1e-4, window)
+        ops.attention_diff_simple(q.float(), want, caches[torch.float32].handles[0].kv, ctx.token_seq, ctx.slots, ctx.positions, *args)
+        out = torch.empty(sum(lens), n_heads * 128, dtype=torch.bfloat16, device=DEV)
+        ops.attention_diff_tcgen05(q, out, caches[torch.bfloat16].handles[0].kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, 5, 700, *args)
+        close(out, f64(want), "bfloat16", (n_heads, size))
     assert ops.bounded_wait_failures() == 0
+
+
+@pytest.mark.parametrize("n_heads,n_kv,d,vd,window", [(8, 2, 64, 128, 0), (16, 1, 64, 128, 0), (4, 4, 32, 64, 100), (12, 2, 128, 256, 0), (3, 1, 24, 40, 64), (6, 2, 128, 64, 1)])
+def test_decode_differential_attention_against_the_plain_kernel(n_heads, n_kv, d, vd, window):
+    """Sequences of one key up to several shares of pages, whole and in shares."""
+    from go_tinygrad_b200.cache import KVRequest
+    rng = np.random.default_rng(d + n_heads)
+    rt = Runtime(DEV, torch.bfloat16)
+    starts = [0, 1, 15, 16, 62, 63, 64, 700, 127, 128]
+    n = len(starts)
+    caches = {}
+    for dt in (torch.bfloat16, torch.float32):
+        c = Cache([[KVRequest(n_kv, 2 * d, None, value_dim=vd)]], [None], max_tokens=64 * 40, max_slots=n, dtype=dt, device=DEV)
+        slots = [c.open_sequence() for _ in range(n)][::-1]
+        c.reserve_many([(s, a + 1) for s, a in zip(slots, starts)]); c.flush_tables()
+        caches[dt] = c
+    store = caches[torch.bfloat16].groups[0].storage
+    store.copy_(t32(rng.standard_normal(tuple(store.shape))).to(torch.bfloat16))
+    caches[torch.float32].groups[0].storage.copy_(store.float())
+    ctx = context(rt, [1] * n, starts, slots)
+    q = (t32(rng.standard_normal((n, n_heads * 2 * d))) * 3).to(torch.bfloat16)
+    want = torch.empty(n, n_heads * vd, dtype=torch.float32, device=DEV)
+    args = (n_heads, d ** -0.5, 0.5, 0.6, 1e-3, window)
+    ops.attention_diff_simple(q.float(), want, caches[torch.float32].handles[0].kv, ctx.token_seq, ctx.slots, ctx.positions, *args)
+    for splits in (1, 2, 3, 12):
+        out = torch.empty(n, n_heads * vd, dtype=torch.bfloat16, device=DEV)
+        scratch = torch.full((int(ops._fn("gtg_attention_diff_scratch_floats")(n, n_heads, vd, splits)) or 1,), float("nan"), dtype=torch.float32, device=DEV)
+        ops.attention_diff_bf16(q, out, caches[torch.bfloat16].handles[0].kv, ctx.cu_seqlens, ctx.slots, ctx.start_pos, n, 1, *args, splits, scratch)
+        close(out, f64(want), "bfloat16", splits)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -395,6 +452,31 @@ def test_a_normed_update_joins_the_hidden_state_which_is_normed_again(dtype):
                     else:
                         assert stream.pending is update and torch.equal(stream.residual, t32(x))       # the wanted rows only: nothing is written back
                         close(got, want[[n - 1, 0]], dtype, (n, h, "rows"))
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("h,top,identities,shared", [(64, 2, True, True), (51, 3, True, False), (2048, 4, False, True), (9000, 1, True, True), (72, 9, True, True)])
+def test_the_norm_that_sums_a_mixtures_rows_itself(dtype, h, top, identities, shared):
+    rng = np.random.default_rng(h)
+    n, rows = 37, 400
+    rt = Runtime(DEV, TORCH[dtype])
+    y, x = t32(rng.standard_normal((rows, h)) * 3), t32(rng.standard_normal((n, h))).to(TORCH[dtype])
+    item_row = rng.integers(-1 if identities else 0, rows, n * top)
+    weights, base = t32(rng.uniform(0.1, 2.0, (n, top))), t32(rng.standard_normal((n, h))) if shared else None
+    update = ops.ExpertSum(y, torch.tensor(item_row, dtype=torch.int32, device=DEV), weights, x if identities else None, base)
+    want = np.zeros((n, h))
+    for t in range(n):
+        for k in range(top):
+            row = item_row[t * top + k]
+            want[t] += float(weights[t, k]) * (f64(y[row]) if row >= 0 else f64(x[t]))
+    want = want + (f64(base) if shared else 0.0)
+    close(update.float(), want, "float32")
+    res, w = rng.standard_normal((n, h)) * 2, [t32(1 + 0.3 * rng.standard_normal(h)) for _ in range(2)]
+    residual, out = t32(res).clone(), torch.empty(n, h, dtype=TORCH[dtype], device=DEV)
+    ops.layernorm_add_layernorm(residual, update, w[0], 1e-5, w[1], None, 1e-5, out)
+    total = f64(t32(res)) + plain.layer_norm(want, f64(w[0]), 1e-5)
+    close(residual, total, "float32")
+    close(out, plain.layer_norm(total, f64(w[1]), 1e-5), dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
