@@ -1367,6 +1367,10 @@ def run_design(args):
                 if not label:
                     base, comb = rnd(n, H, dtype=f32), torch.empty(n, H, dtype=f32, device=dev)
                     ops.moe_product(act, row_item, 0, w_dn, tile_e, yy)
+                    mix = ops.ExpertSum(yy, item_row, weights, x, base)
+                    mix_bytes = real * H * 4 + (n * top - real) * H * 2 + n * H * 4
+                    add(f"layernorm_add_layernorm, summing a mixture ({tag})", n,
+                        timed(lambda: ops.layernorm_add_layernorm(res, mix, w, 1e-5, w, None, 1e-5, out)), mix_bytes + n * H * (4 + 4 + 2))
                     add(f"moe_combine, identities and shared ({tag})", n, timed(lambda: ops.moe_combine(yy, item_row, weights, comb, x=x, base=base)),
                         real * H * 4 + (n * top - real) * H * 2 + n * H * 8)
                 else:
