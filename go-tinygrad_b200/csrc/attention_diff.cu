@@ -719,8 +719,9 @@ GTG_API long long gtg_attention_diff_scratch_floats(int n_tokens, int n_heads, i
     return (long long)n_tokens * n_heads * 2 * n_splits * (padded(vd) + 2);
 }
 
-// Into how many shares the pages of a step's tiles are cut: 1 while the tiles alone fill the device;
-// else as many as bring about two blocks per multiprocessor, each share two pages at least.
+// Into how many shares the pages of a step's tiles are cut: the number for which the waves of blocks (two to a
+// multiprocessor) times the pages a block walks, plus what a block costs beyond its pages, is least; a second kernel
+// merges the shares, which counts too.  It depends on the step's sizes only.
 GTG_API int gtg_attention_diff_splits(int n_seqs, int max_q_len, int n_heads, int n_kv, int max_kv_len, int window) {
     if (n_seqs <= 0 || n_kv <= 0) return 1;
     int device = 0, sms = 148;
@@ -729,9 +730,15 @@ GTG_API int gtg_attention_diff_splits(int n_seqs, int max_q_len, int n_heads, in
     const long long blocks = tiles * n_kv * n_seqs;
     const int keys = window > 0 ? min(max_kv_len, window + max_q_len) : max_kv_len;
     const int pages = (keys + kPageTokens - 1) / kPageTokens + (window > 0 ? 1 : 0);
-    if (blocks >= 2LL * sms || pages < 4) return 1;
-    const long long want = min((2LL * sms + blocks - 1) / blocks, (long long)pages / 2);
-    return (int)max(1LL, min(want, 32LL));
+    constexpr long long kBlockPages = 2, kMergePages = 4;  // a block's start and end, and the merge, in pages' time
+    int best = 1;
+    long long least = -1;
+    for (int n = 1; n <= min(32, pages); ++n) {
+        const long long waves = (blocks * n + 2LL * sms - 1) / (2LL * sms);
+        const long long cost = waves * ((pages + n - 1) / n + kBlockPages) + (n > 1 ? kMergePages : 0);
+        if (least < 0 || cost < least) { least = cost; best = n; }
+    }
+    return best;
 }
 
 GTG_API int gtg_attention_diff_bf16(const void* q, int ldq, void* out, int ldo, const void* kc, const void* vc,

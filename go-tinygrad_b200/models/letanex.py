@@ -90,4 +90,5 @@ LETANEX = register_architecture(Architecture(
     names=("Letanex", "letanex"),
     read_config=LetanexConfig.from_json,
     plan=letanex_plan,
+    ignore=("l*.norm2", "l*.norm2b"),      # a layer without a feed-forward may carry the norms of one
 ))
