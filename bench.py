@@ -553,7 +553,7 @@ def letanex_shape(width, heads, kv_heads, ff, experts, expert_ff, top, vocab=320
     att = {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
            "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 4.0}}}
     routed = {"kind": "moe", "expert": {"ff": expert_ff, "limit": 7.0}, "shared": {"ff": expert_ff, "limit": 7.0},
-              "router": {"experts": experts, "top": top, "identity": 4, "scale": 1.5}}
+              "router": {"experts": experts, "top": top, "identity": 4, "scale": 2.0}}
     layers = []
     for i in range(8):
         mixer = light if i % 2 == 0 else dict(att, kv_from=i - 2) if i % 4 == 3 else att

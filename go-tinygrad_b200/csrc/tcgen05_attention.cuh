@@ -19,7 +19,6 @@ template <bool kTest> struct Waits {
 };
 static bool g_test_waits = false;       // set by the test hook: launches take the kTest form
 
-
 __device__ int g_status = 0;
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }

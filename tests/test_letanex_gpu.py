@@ -46,8 +46,8 @@ CONFIG_Q = {
     "architecture": "Letanex", "vocab": 160, "width": 128, "norm": {"eps": 1e-6},
     "layers": [
         lightning([0.6, 0.95, 0.995, 0.999], 64, 128, dense(256)),
-        attention(4, 1, 64, 128, 0.12, 0.35, rotation(64, 10000.0, 8.0), moe(64, 2.0, 8, 2, 2, 1.5, (128, 1.5))),
-        attention(4, 1, 64, 128, 0.12, 0.3, rotation(64, 10000.0, 8.0), moe(64, 2.0, 8, 2, 2, 1.5, (128, 1.5)), kv_from=1),
+        attention(4, 1, 64, 128, 0.12, 0.35, rotation(64, 10000.0, 6.0), moe(64, 1.8, 8, 2, 2, 1.4, (128, 1.3))),
+        attention(4, 1, 64, 128, 0.12, 0.3, rotation(64, 10000.0, 6.0), moe(64, 1.8, 8, 2, 2, 1.4, (128, 1.3)), kv_from=1),
         attention(2, 2, 128, 256, 0.09, 0.4, rotation(32, 500.0, 4.0), None),
         lightning([0.8, 0.9995], 128, 64, moe(128, 1.0, 4, 4, 4, 1.0, (64, 2.5))),
     ],
@@ -189,7 +189,7 @@ CUTS = lambda T: ([T], [1] * T, [2] * (T // 2), [63, 1, 1, 64, T - 129], [T - 50
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,dims,factor", [
-    (4, 2, 16, 24, 8, 4.0), (3, 1, 5, 7, 4, None), (6, 6, 8, 8, 8, 1.5), (2, 1, 64, 128, 64, 8.0), (8, 2, 64, 64, 32, 2.0), (5, 1, 24, 48, None, None),
+    (4, 2, 16, 24, 8, 4.0), (3, 1, 5, 7, 4, None), (6, 6, 8, 8, 8, 1.5), (2, 1, 64, 128, 64, 7.0), (8, 2, 64, 64, 32, 2.0), (5, 1, 24, 48, None, None),
     (1, 1, 80, 40, 16, 3.0), (2, 2, 128, 256, 128, None), (4, 1, 128, 128, 64, 2.0), (16, 1, 32, 64, 32, 1.0), (3, 3, 40, 160, 10, 2.0)])
 def test_differential_attention_with_keys_of_its_own_and_borrowed(dtype, heads, kv_heads, dim, vdim, dims, factor):
     """Random weights, two layers over one cache; scores large enough that a key, a map, a rotation or a lambda that is
