@@ -21,8 +21,8 @@ namespace {
 // The columns of S never meet.  One block serves (head, a slice of columns, sequence); R lanes of a warp
 // share a column, lane r owning rows r, r + R, ... (up to kRows of them) in registers; their partial sums
 // meet by shuffles.  q, k and v of a tile of tokens at a time are staged in shared memory as floats.
-// Tokens are walked strictly in order: the result does
-// not depend on the cut of the sequence into steps, on the batch or on the slices.
+// Tokens are walked strictly in order: the result does not depend on the cut of the sequence into steps, on
+// the batch or on the slices.
 constexpr int kRows = 16;
 constexpr int kScanThreads = 128;
 constexpr int kTile = 8;

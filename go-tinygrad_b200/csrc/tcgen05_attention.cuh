@@ -12,7 +12,7 @@ constexpr unsigned kSpinLimit = 1u << 22;
 // test of the give-up path launches, whose waits poll a thousand times instead of
 // millions and whose asynchronous copies are not issued at all, so that every
 // barrier it waits on never completes.  The second form is the first form's code
-// with these two constants changed; see the test hook at the end of this file.
+// with these two constants changed; see the test hook at the end of the library's own file.
 template <bool kTest> struct Waits {
     static constexpr unsigned kLimit = kTest ? 1024u : kSpinLimit;
     static constexpr bool kSkipCopies = kTest;
